@@ -5,3 +5,4 @@ from .turevik import TurevikConfig  # noqa: F401
 from .porarax import PoraraxConfig  # noqa: F401
 from .sogazen import SogazenConfig  # noqa: F401
 from .kimutar import KimutarConfig  # noqa: F401
+from .kefetar import KefetarConfig  # noqa: F401

@@ -400,6 +400,39 @@ int tlc_wkv_scan(const float* rkv, int ld, int r_off, int k_off, int v_off, cons
                  const float* bonus, float* state, const int* cu_seqlens, const int* slots, const int* start_pos, int B,
                  int H, int d, float* out, int out_ld, cudaStream_t stream);
 
+/* ---- short linear convolutions over time (short_conv.cu) -----------------------------------------------------
+ * tlc_rmsnorm_conv: h = x / sqrt(mean(x^2) + eps) * g, out[t] = h[t] + sum_j w[j] * h[t - K + 1 + j] (zeros before a sequence's
+ * first row); x float [T, D], g [D], w [K, D]; the last K - 1 rows h of a sequence are kept in state float [n_slots, K - 1, D].
+ * tlc_channel_conv: y[t] = sum_j w[j] * u[t - K + 1 + j] for the C columns of proj float [T, ld] from `off`, w [K, C], state float
+ * [n_slots, K - 1, C], out float [T, C]; with `first` (float [T, ld_first], or NULL) the columns from mix_from on,
+ * heads of hd columns that hold vd values, become (1 - lam) * y + lam * first[t, .] value by value, the rows of `first` holding as
+ * many values in heads of vd_first in hd_first columns.  single_rows: row b is sequence b's only one; all_fresh: every sequence
+ * starts at position 0. */
+int tlc_rmsnorm_conv(const float* x, const float* g, float eps, const float* w, float* state, const int* cu_seqlens,
+                     const int* row_seq, const int* slots, const int* start_pos, void* out, int out_dtype, int T, int B, int D,
+                     int K, int single_rows, int all_fresh, cudaStream_t stream);
+int tlc_channel_conv(const float* proj, int ld, int off, const float* w, float* state, const int* cu_seqlens, const int* row_seq,
+                     const int* slots, const int* start_pos, float* out, const float* first, int ld_first, int mix_from, int hd,
+                     int vd, int hd_first, int vd_first, float lam, int T, int B, int C, int K, int single_rows, int all_fresh,
+                     cudaStream_t stream);
+
+/* ---- polynomial activation over normed powers (polynorm.cu) -----------------------------------------------------
+ * out = a N(z) + b N(z^2) + c N(z^3) + e with N(u) = u / sqrt(mean(u^2) + eps) over a row of F values; z float [T, ldz]. */
+int tlc_polynorm(const float* z, int ldz, int T, int F, float a, float b, float c, float e, float eps, void* out, int dtype,
+                 cudaStream_t stream);
+
+/* ---- retention (retention.cu) ------------------------------------------------------------------------------------
+ * Per head S <- a S + k v^T, o = S^T q, with q and k rotated (split halves of the first rope_dim dimensions) and k times
+ * k_scale; state float [n_slots, H, dv, dk] (zero at position 0).  tlc_retention_prepare lays prompt rows out for the
+ * selective scan: vkq [T, H * dv | H * dk | H * dk], ones and decays [T, H].  tlc_retention_decode: one row per sequence,
+ * out = o / sqrt(mean(o^2) + eps) * silu(gate), head by head. */
+int tlc_retention_prepare(const float* proj, int ld, int q_off, int k_off, int v_off, const float* inv_freq, int rope_dim,
+                          const int* positions, const float* decay, float k_scale, int T, int H, int dk, int dv, float* vkq,
+                          float* ones, float* decays, cudaStream_t stream);
+int tlc_retention_decode(const float* proj, int ld, int q_off, int k_off, int v_off, int g_off, const float* inv_freq, int rope_dim,
+                         const int* positions, const int* slots, const float* decay, float k_scale, float eps, float* state, int B,
+                         int H, int dk, int dv, void* out, int out_dtype, int out_ld, cudaStream_t stream);
+
 /* ---- sampling (sampling.cu) ------------------------------------------------------------------------ */
 /* out[r] = first index of the maximum of logits[r].  work: NULL (one block a row), or 12 * R bytes, 8-byte
  * aligned and zero (R 64-bit keys, R counters), which every launch leaves zero: a row is then spread over

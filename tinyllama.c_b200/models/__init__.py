@@ -4,3 +4,4 @@ from . import turevik  # noqa: F401  (registers Turevik)
 from . import porarax  # noqa: F401  (registers Porarax)
 from . import sogazen  # noqa: F401  (registers Sogazen)
 from . import kimutar  # noqa: F401  (registers Kimutar)
+from . import kefetar  # noqa: F401  (registers Kefetar)

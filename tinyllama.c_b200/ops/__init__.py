@@ -101,6 +101,11 @@ _SIGNATURES = {
     "tlc_qk_whole_norm": (_i, [_vp, _i, _i, _i, _vp, _i, _i, _vp, _f, _i, _vp]),
     "tlc_shift_mix": (_i, [_vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp]),
     "tlc_wkv_scan": (_i, [_vp, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _vp]),
+    "tlc_rmsnorm_conv": (_i, [_vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]),
+    "tlc_channel_conv": (_i, [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _i, _i, _vp]),
+    "tlc_polynorm": (_i, [_vp, _i, _i, _i, _f, _f, _f, _f, _f, _vp, _i, _vp]),
+    "tlc_retention_prepare": (_i, [_vp, _i, _i, _i, _i, _vp, _i, _vp, _vp, _f, _i, _i, _i, _i, _vp, _vp, _vp, _vp]),
+    "tlc_retention_decode": (_i, [_vp, _i, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _f, _f, _vp, _i, _i, _i, _i, _vp, _i, _i, _vp]),
     "tlc_moe_identity": (_i, [_vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _vp, _vp]),
     "tlc_rmsnorm_shift": (_i, [_vp, _vp, _vp, _f, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp]),
     "tlc_rmsnorm_add": (_i, [_vp, _i, _vp, _vp, _i, _i, _vp, _f, _i, _i, _vp, _i, _vp, _i, _vp]),
@@ -1339,3 +1344,122 @@ def delta_rule(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, beta: torc
     _call("tlc_delta_rule", qkv.data_ptr(), _rows(qkv, "qkv"), int(q_off), int(k_off), int(v_off), beta.data_ptr(), decay.data_ptr(),
           state.data_ptr(), step.cu_seqlens.data_ptr(), step.slots.data_ptr(), step.start_pos.data_ptr(), step.n_seqs, T, int(H),
           int(G), int(dk), int(dv), y.data_ptr(), ldy, _rows(decay, "decays") if per_channel else 0, _stream())
+
+
+# ---- short linear convolutions over time ----------------------------------------------------------------------
+def _all_fresh(step) -> int:
+    """Whether every sequence of the step starts at position 0 (known on the host)."""
+    return int(len(step.host_start) == step.n_seqs and not any(step.host_start))
+
+
+def _window(state: Optional[torch.Tensor], K: int, C: int, what: str) -> Optional[int]:
+    if K == 1:
+        return None
+    if state is None or state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (K - 1, C):
+        raise KernelError(f"{what}: the kept rows must be contiguous float32 [n_slots, {K - 1}, {C}]")
+    return state.data_ptr()
+
+
+def rmsnorm_conv(x: torch.Tensor, weight: torch.Tensor, eps: float, taps: torch.Tensor, state: Optional[torch.Tensor], step,
+                 out: torch.Tensor) -> None:
+    """h = rmsnorm(x) * weight; out[t] = h[t] + sum_j taps[j] * h[t - K + 1 + j] (zeros before a sequence's first row): x float32
+    [T, D], taps float32 [K, D], state float32 [n_slots, K - 1, D] (a sequence's last K - 1 rows h, updated in place; None
+    with one tap)."""
+    _gpu(x, weight, taps, state, out)
+    T, D = x.shape
+    K = taps.shape[0]
+    if x.dtype != torch.float32 or not x.is_contiguous() or not out.is_contiguous() or tuple(out.shape) != (T, D):
+        raise KernelError("rmsnorm_conv: x must be contiguous float32 [T, D] and out contiguous [T, D]")
+    _f32vec(weight, D, "rmsnorm_conv weight")
+    _f32vec(taps, K * D, "rmsnorm_conv taps")
+    _call("tlc_rmsnorm_conv", x.data_ptr(), weight.data_ptr(), float(eps), taps.data_ptr(), _window(state, K, D, "rmsnorm_conv"),
+          step.cu_seqlens.data_ptr(), step.row_seq.data_ptr(), step.slots.data_ptr(), step.start_pos.data_ptr(), out.data_ptr(),
+          dtype_code(out.dtype), T, step.n_seqs, D, K, int(step.max_new == 1), _all_fresh(step), _stream())
+
+
+def channel_conv(proj: torch.Tensor, off: int, taps: torch.Tensor, state: Optional[torch.Tensor], step, out: torch.Tensor,
+                 first: Optional[torch.Tensor] = None, mix_from: int = 0, lam: float = 0.0, heads=(1, 1), first_heads=None) -> None:
+    """out[t, c] = sum_j taps[j, c] * proj[t - K + 1 + j, off + c] within each sequence (zeros before its first row): proj
+    float32 [T, *], taps float32 [K, C], out contiguous float32 [T, C], state as in rmsnorm_conv.  first (float32 [T, *],
+    dense rows): the columns from mix_from on become (1 - lam) * y + lam * first[t, .], value by value; heads = (columns of a
+    head, values in it) of these columns, first_heads the same of first's (default: one layout)."""
+    _gpu(proj, taps, state, out, first)
+    T = proj.shape[0]
+    K, C = taps.shape
+    ld = _rows(proj, "channel_conv input")
+    if proj.dtype != torch.float32 or out.dtype != torch.float32 or not out.is_contiguous() or tuple(out.shape) != (T, C) \
+            or off + C > max(ld, proj.shape[1]):
+        raise KernelError("channel_conv: a float32 projection that holds the columns, out contiguous float32 [T, C]")
+    _f32vec(taps, K * C, "channel_conv taps")
+    hd, vd = heads
+    hd_f, vd_f = first_heads or heads
+    if first is not None and (first.dtype != torch.float32 or first.shape[0] != T or hd < 1
+                              or first.shape[1] // hd_f * vd_f != (C - mix_from) // hd * vd):
+        raise KernelError(f"channel_conv: what is blended in must be float32 rows of as many values as the {C - mix_from} columns hold")
+    _call("tlc_channel_conv", proj.data_ptr(), ld, int(off), taps.data_ptr(), _window(state, K, C, "channel_conv"),
+          step.cu_seqlens.data_ptr(), step.row_seq.data_ptr(), step.slots.data_ptr(), step.start_pos.data_ptr(), out.data_ptr(), _p(first),
+          0 if first is None else _rows(first, "channel_conv blend"), int(mix_from), int(hd), int(vd), int(hd_f), int(vd_f), float(lam), T,
+          step.n_seqs, C, K, int(step.max_new == 1), _all_fresh(step), _stream())
+
+
+def polynorm(z: torch.Tensor, coefficients, eps: float, out: torch.Tensor) -> None:
+    """out = a N(z) + b N(z^2) + c N(z^3) + e, N(u) = u / sqrt(mean(u^2) + eps) over a row; z float32 [T, F], out contiguous."""
+    _gpu(z, out)
+    T, F = z.shape
+    if z.dtype != torch.float32 or not out.is_contiguous() or tuple(out.shape) != (T, F):
+        raise KernelError("polynorm: z float32 [T, F] and out contiguous [T, F]")
+    a, b, c, e = [float(v) for v in coefficients]
+    _call("tlc_polynorm", z.data_ptr(), _rows(z, "polynorm input"), T, F, a, b, c, e, float(eps), out.data_ptr(), dtype_code(out.dtype),
+          _stream())
+
+
+# ---- retention ------------------------------------------------------------------------------------------------
+MAX_RETENTION_KEY_DIM = 256      # retention.cu, mamba.cu: key columns of a head's state that a warp holds in registers
+MAX_RETENTION_VALUE_DIM = 4096   # retention.cu: values of a head in shared memory
+
+
+def _retention_checks(proj, inv_freq, decay, state, H, dk, dv, offsets, what):
+    _gpu(proj, inv_freq, decay, state)
+    ld = _rows(proj, what + " projection")
+    if proj.dtype != torch.float32 or any(o + n > max(ld, proj.shape[1]) for o, n in offsets):
+        raise KernelError(f"{what}: a float32 projection that holds every head")
+    _f32vec(inv_freq, inv_freq.numel(), "rotation inv_freq")
+    _f32vec(decay, H, what + " decays")
+    if state is not None and (state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (H, dv, dk)):
+        raise KernelError(f"{what}: the state must be contiguous float32 [n_slots, H, dv, dk]")
+    return ld
+
+
+def retention_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, inv_freq: torch.Tensor, positions: torch.Tensor,
+                      decay: torch.Tensor, k_scale: float, H: int, dk: int, dv: int, vkq: torch.Tensor, ones: torch.Tensor,
+                      decays: torch.Tensor) -> None:
+    """Lays prompt rows out as the selective scan (ssm_scan) reads them: vkq float32 [T, H*dv | H*dk | H*dk] holds the values,
+    the rotated keys times k_scale and the rotated queries; ones and decays float32 [T, H] are the scan's step sizes and
+    factors."""
+    ld = _retention_checks(proj, inv_freq, decay, None, H, dk, dv, ((q_off, H * dk), (k_off, H * dk), (v_off, H * dv)), "retention_prepare")
+    _gpu(vkq, ones, decays)
+    _i32(positions, "positions")
+    T = proj.shape[0]
+    for t, shape in ((vkq, (T, H * (dv + 2 * dk))), (ones, (T, H)), (decays, (T, H))):
+        if t.dtype != torch.float32 or not t.is_contiguous() or tuple(t.shape) != shape:
+            raise KernelError(f"retention_prepare: results must be contiguous float32 {shape}")
+    _call("tlc_retention_prepare", proj.data_ptr(), ld, int(q_off), int(k_off), int(v_off), inv_freq.data_ptr(), 2 * inv_freq.numel(),
+          positions.data_ptr(), decay.data_ptr(), float(k_scale), T, int(H), int(dk), int(dv), vkq.data_ptr(), ones.data_ptr(),
+          decays.data_ptr(), _stream())
+
+
+def retention_decode(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, inv_freq: torch.Tensor, decay: torch.Tensor,
+                     k_scale: float, eps: float, state: torch.Tensor, step, H: int, dk: int, dv: int, out: torch.Tensor) -> None:
+    """One-token steps: per head S <- a S + k v^T, o = S^T q (q, k rotated at the row's position, k times k_scale), out = o /
+    sqrt(mean(o^2) + eps) * silu(gate); proj float32 [B, *] holds q, k, v and the gate; state float32 [n_slots, H, dv, dk]
+    (zero at position 0; updated in place); out [B, H*dv]."""
+    ld = _retention_checks(proj, inv_freq, decay, state, H, dk, dv, ((q_off, H * dk), (k_off, H * dk), (v_off, H * dv), (g_off, H * dv)),
+                           "retention_decode")
+    _gpu(out)
+    B = proj.shape[0]
+    if step.n_seqs != B:
+        raise KernelError("retention_decode: one row per sequence")
+    _call("tlc_retention_decode", proj.data_ptr(), ld, int(q_off), int(k_off), int(v_off), int(g_off), inv_freq.data_ptr(),
+          2 * inv_freq.numel(), step.positions.data_ptr(), step.slots.data_ptr(), decay.data_ptr(), float(k_scale), float(eps),
+          state.data_ptr(), B, int(H), int(dk), int(dv), out.data_ptr(), dtype_code(out.dtype), _out_rows(out, B, H * dv, "retention_decode"),
+          _stream())

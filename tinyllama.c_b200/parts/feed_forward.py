@@ -77,25 +77,36 @@ class SwiGLU(Part):
 
 @register_feed_forward("mlp")
 class DenseFeedForward(Part):
-    """A feed-forward without a gate: d = W_down act(W_up x), act the square of max(., 0) ("relu_squared").  Two products
-    with the activation between them (32-bit in, activation type out)."""
+    """A feed-forward without a gate: d = W_down act(W_up x), act the square of max(., 0) ("relu_squared") or a polynomial
+    over normed powers of the token's whole row ("polynorm"): a N(z) + b N(z^2) + c N(z^3) + e with N(u) = u / sqrt(mean(u^2) +
+    eps) and four learned numbers.  Two products with the activation between them (32-bit in, activation type out)."""
 
-    def __init__(self, hidden: int, intermediate: int, names: Dict[str, str], act: str = "relu_squared"):
-        """names: tensor names of up and down."""
-        if act not in ("relu_squared",):
-            raise ValueError(f"feed-forward: unknown activation '{act}' of a feed-forward without a gate; known: ['relu_squared']")
-        self.hidden, self.F, self.act = int(hidden), int(intermediate), act
+    def __init__(self, hidden: int, intermediate: int, names: Dict[str, str], act: str = "relu_squared", act_eps: float = 0.0):
+        """names: tensor names of up and down; with act "polynorm" also act, the tensor of a, b, c, e.  act_eps: under the
+        roots of "polynorm"."""
+        if act not in self.ACTS:
+            raise ValueError(f"feed-forward: unknown activation '{act}' of a feed-forward without a gate; known: {list(self.ACTS)}")
+        if act == "polynorm" and not (act_eps > 0 and "act" in names):
+            raise ValueError("feed-forward: the polynomial activation needs the name of its numbers ('act') and a positive act_eps")
+        self.hidden, self.F, self.act, self.act_eps = int(hidden), int(intermediate), act, float(act_eps)
+        self.act_name = names["act"] if act == "polynorm" else None
+        self.coefficients = None
         self.up = StackedLinear(hidden)
         self.up.add(names["up"], self.F)
         self.down = StackedLinear(self.F)
         self.down.add(names["down"], hidden)
 
+    ACTS = ("relu_squared", "polynorm")
+
     def weight_specs(self) -> List[WeightSpec]:
-        return self.up.weight_specs() + self.down.weight_specs()
+        own = [WeightSpec(self.act_name, (4,), "unit_interval")] if self.act_name else []
+        return self.up.weight_specs() + self.down.weight_specs() + own
 
     def bind(self, tensors: Dict[str, torch.Tensor], dtype, device) -> None:
         self.up.bind(tensors, dtype, device)
         self.down.bind(tensors, dtype, device)
+        if self.act_name:
+            self.coefficients = tuple(float(v) for v in tensors[self.act_name].to(device="cpu", dtype=torch.float32))
 
     def forward(self, normed: torch.Tensor, residual: torch.Tensor, accumulate: bool = True) -> None:
         """Adds the result into `residual` (float32 [T, D]), or overwrites it with accumulate False."""
@@ -103,7 +114,10 @@ class DenseFeedForward(Part):
         u = scratch_buf("mlp.up", (T, self.F), torch.float32, normed.device)
         self.up.forward(normed, u)
         act = scratch_buf("mlp.act", (T, self.F), normed.dtype, normed.device)
-        ops.convert(u, act, self.act)
+        if self.act == "polynorm":
+            ops.polynorm(u, self.coefficients, self.act_eps, act)
+        else:
+            ops.convert(u, act, self.act)
         self.down.forward(act, residual, accumulate=accumulate)
 
     def forward_parts(self, normed: torch.Tensor):

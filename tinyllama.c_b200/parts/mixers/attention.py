@@ -20,6 +20,9 @@ heads, one for all key heads); frequencies stretched for long sequences and cosi
 position part's business); a sink whose score is learned per head; a window that keeps the sequence's first keys visible;
 and two score maps per head over the same values whose results are subtracted and normed (`maps=2`): the kernels then see
 twice the heads, the queries regrouped so that a map's heads share the map's keys, and one kernel joins the pairs.
+And: a short causal convolution over time on every channel of the projected q, k and v, before any norm or rotation (the
+last taps - 1 projected rows of a sequence are kept between steps); and values blended with those of another layer, the
+first of the layers that share them, of the same token: v <- (1 - lam) v + lam v_first.
 """
 from __future__ import annotations
 
@@ -29,7 +32,7 @@ from typing import Dict, List, Optional
 import torch
 
 from ... import ops
-from ..base import KVRequest, LayerCache, Part, PartSpec, StepInfo, WeightSpec, act_empty, register_mixer, scratch_buf, to_vec
+from ..base import KVRequest, LayerCache, Part, PartSpec, StateRequest, StepInfo, WeightSpec, act_empty, register_mixer, scratch_buf, to_vec
 from ..linear import StackedLinear
 
 
@@ -42,7 +45,8 @@ class AttentionMixer(Part):
                  qk_norm_eps: Optional[float] = None, gate: Optional[str] = None, values: str = "projection",
                  whole_norm: Optional[Dict[str, object]] = None, softcap: float = 0.0, sink: bool = False,
                  head_norm: Optional[Dict[str, object]] = None, sink_name: Optional[str] = None, keep_first: int = 0,
-                 maps: int = 1, difference: Optional[Dict[str, object]] = None):
+                 maps: int = 1, difference: Optional[Dict[str, object]] = None, conv_taps: int = 0,
+                 v_mix: Optional[Dict[str, object]] = None):
         """names: tensor names of q, k, v, o (and g, the gate's projection) after the prefix, where they are not the
         q_proj.weight ... of the architecture's checkpoints (biases then take no part).  scale: what scores are
         multiplied by (default head_dim ** -0.5).  v_dim: size of a value head (default head_dim).  qk_norm_eps: queries
@@ -58,7 +62,11 @@ class AttentionMixer(Part):
         maps = 2 with difference = dict(init=number, eps=..., lq1=, lk1=, lq2=, lk2= names of vectors [head_dim]): the q tensor
         has n_heads * 2 * head_dim rows and the k tensor n_kv_heads * 2 * head_dim, head by head as [map 1, map 2]; each map is
         an attention of its own over the head's values, and with lam = exp(lq1 . lk1) - exp(lq2 . lk2) + init the head's result
-        is o = a1 - lam a2, o / sqrt(mean(o^2) + eps) * (1 - init)."""
+        is o = a1 - lam a2, o / sqrt(mean(o^2) + eps) * (1 - init).  conv_taps > 0: tensors named q, k, v + ".conv" ([channels,
+        taps], newest tap last) smooth the projected q, k and v along the sequence, y_t = sum_j w[:, j] u_(t - taps + 1 + j),
+        before anything else.  v_mix (with conv_taps) = dict(group=any name, first=True) for the layer whose (convolved) values
+        the later ones of the group take a share of, dict(group=..., name=tensor of one number lam) for those:
+        v <- (1 - lam) v + lam v_first; the blended v is what is cached."""
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} heads are not a multiple of {n_kv_heads} key/value heads")
         if not (1 <= int(head_dim) <= ops.MAX_HEAD_DIM):
@@ -94,7 +102,7 @@ class AttentionMixer(Part):
         if self.head_norm and not {"q", "k", "eps"} <= set(self.head_norm):
             raise ValueError("attention: a norm per head needs q, k (weight names) and eps")
         self.pre_transform = layout == "interleaved" or self.qk_norm_eps is not None or self.head_norm is not None \
-            or getattr(self.position, "scaling", None) is not None
+            or (getattr(self.position, "scaling", None) or {}).get("kind") in ("bands", "ramp")
         if names is not None and bias:
             raise ValueError("attention: tensor names of one's own name their biases themselves (q_bias, k_bias, v_bias)")
         if values not in ("projection", "keys"):
@@ -143,6 +151,20 @@ class AttentionMixer(Part):
         self.dtype = None
         self.prefix = prefix
         self.q_norm_w = self.k_norm_w = None
+        # the convolution runs over the stacked q | k | v columns of the projection: its weights are laid out like them
+        self.conv_taps = int(conv_taps)
+        self.v_mix = dict(v_mix) if v_mix else None
+        if self.conv_taps and not (1 <= self.conv_taps <= ops.MAX_CONV_TAPS):
+            raise ValueError(f"attention: {conv_taps} convolution taps are outside what the kernels are built for (1..{ops.MAX_CONV_TAPS})")
+        if self.conv_taps and (self.maps > 1 or values != "projection"):
+            raise ValueError("attention: a convolution of q, k and v goes with one map and values of their own")
+        if self.v_mix and (not self.conv_taps or "group" not in self.v_mix or bool(self.v_mix.get("first")) == ("name" in self.v_mix)):
+            raise ValueError("attention: blended values go with a convolution and need a group and either first=True or the name of their share")
+        self.conv_channels = (self.H + 2 * self.KV) * self.hd
+        self.conv_parts = [(prefix + nm[n] + ".conv", heads, dim) for n, heads, dim in
+                           (("q", self.H, self.qk_dim), ("k", self.KV, self.qk_dim), ("v", self.KV, self.v_dim))] if self.conv_taps else []
+        self.conv_w = None
+        self.mix_share = 0.0
 
     @property
     def single_token_launches(self) -> int:
@@ -177,10 +199,16 @@ class AttentionMixer(Part):
             specs.append(WeightSpec(self.prefix + self.sink_name, (self.Hq,), "near_zero"))
         if self.difference:
             specs += [WeightSpec(self.prefix + self.difference[n], (self.qk_dim,), "near_zero") for n in ("lq1", "lk1", "lq2", "lk2")]
+        specs += [WeightSpec(name, (heads * dim, self.conv_taps), "conv") for name, heads, dim in self.conv_parts]
+        if self.v_mix and "name" in self.v_mix:
+            specs.append(WeightSpec(self.prefix + str(self.v_mix["name"]), (), "unit_interval"))
         return specs
 
     def cache_requests(self) -> list:
-        return [KVRequest(self.cache_key, self.KV, self.hd, self.window, keep_first=self.keep_first if self.window else 0)]
+        reqs = [KVRequest(self.cache_key, self.KV, self.hd, self.window, keep_first=self.keep_first if self.window else 0)]
+        if self.conv_taps > 1:
+            reqs.append(StateRequest(self.cache_key + ".conv", (self.conv_taps - 1, self.conv_channels)))
+        return reqs
 
     def bind(self, tensors: Dict[str, torch.Tensor], dtype, device) -> None:
         self.dtype = dtype
@@ -200,6 +228,16 @@ class AttentionMixer(Part):
             vec = lambda n: tensors[self.prefix + self.difference[n]].to(device="cpu", dtype=torch.float32)
             init = float(self.difference["init"])
             self.lam = float(torch.exp((vec("lq1") * vec("lk1")).sum()) - torch.exp((vec("lq2") * vec("lk2")).sum())) + init
+        if self.conv_taps:               # tap by tap, [taps, q | k | v] with zeros where heads are padded
+            rows = []
+            for name, heads, dim in self.conv_parts:
+                w = tensors[name].to(device=device, dtype=torch.float32)
+                full = torch.zeros((heads, self.hd, self.conv_taps), dtype=torch.float32, device=device)
+                full[:, :dim] = w.reshape(heads, dim, self.conv_taps)
+                rows.append(full.reshape(heads * self.hd, self.conv_taps))
+            self.conv_w = torch.cat(rows, dim=0).t().contiguous()
+        if self.v_mix and "name" in self.v_mix:
+            self.mix_share = float(tensors[self.prefix + str(self.v_mix["name"])].to(torch.float32).reshape(-1)[0])
         self._no_rotation = torch.zeros(0, dtype=torch.float32, device=device)
         # arrival counters of the one-kernel attention of single-token steps: this mixer's own, so that no other
         # mixer, model or stream ever shares them; made here, outside any stream capture
@@ -233,6 +271,9 @@ class AttentionMixer(Part):
         holds at most that many SMs (a block that runs another mixer beside this one leaves it the rest)."""
         T = step.n_rows
         kv = cache.kv[self.cache_key]
+        projected = qkv                    # (the gate's columns stay there)
+        if self.conv_taps:
+            qkv = self._convolved(qkv, step, cache)
         if self.whole_norm:           # over all heads at once, before any rotation (the value columns keep the projection)
             ops.qk_whole_norm(qkv, self.q_off, self.H * self.hd, self.q_norm_w, self.k_off, self.KV * self.hd, self.k_norm_w,
                               float(self.whole_norm["eps"]))
@@ -257,7 +298,7 @@ class AttentionMixer(Part):
                                        cache.writes, kv.block_table, step.positions, step.row_seq, step.slots, att,
                                        self.H, self.KV, self.hd, self.scale, self.window or 0,
                                        step.max_context, self._arrivals, self.softcap, self.sink, self.keep_first, self.sink_values)
-            return self._joined(self._gated(att, qkv), joined)
+            return self._joined(self._gated(att, projected), joined)
         q = scratch_buf(f"attention.{self.cache_key}.q", (T, self.H * self.hd), self.dtype, qkv.device)
         ops.rope_kv_store(qkv, self.q_off, self.k_off, self.v_off, q, kv.k_pages, kv.v_pages, table, step.positions,
                           step.row_seq, step.slots, kv.block_table, self.H, self.KV, self.hd, cache.writes)
@@ -266,7 +307,29 @@ class AttentionMixer(Part):
                       self.H, self.KV, self.hd, self.scale, self.window or 0,
                       step.max_context if step.max_new == 1 else 0, step.cu_seqlens, step.start_pos, step.max_context,
                       max_blocks, softcap=self.softcap, sink=self.sink, keep_first=self.keep_first, sink_values=self.sink_values)
-        return self._joined(self._gated(att, qkv), joined)
+        return self._joined(self._gated(att, projected), joined)
+
+    def _convolved(self, qkv: torch.Tensor, step: StepInfo, cache: LayerCache) -> torch.Tensor:
+        """The convolved q | k | v columns, the values blended with the group's first layer's, float32 [T, q | k | v].  The first
+        layer's buffer lives until the step ends (later layers read its values there)."""
+        if not (cache.writes and cache.kv_writes):
+            raise ValueError("attention: a convolution of q, k and v cannot run on another layer's cache without storing "
+                             "(its kept rows would advance twice in one step)")
+        mix = self.v_mix
+        lead = bool(mix and mix.get("first"))
+        tag = f"attention.first.{mix['group']}" if lead else f"attention.{self.cache_key}.convolved"
+        out = scratch_buf(tag, (step.n_rows, self.conv_channels), torch.float32, qkv.device)
+        first, heads = None, (self.hd, self.v_dim)
+        first_heads = heads
+        if mix and not lead:
+            first, first_heads = step.scratch.get(("attention.values", mix["group"]), (None, None))
+            if first is None:
+                raise ValueError(f"attention: no layer of this step has left the values that group '{mix['group']}' blends with")
+        ops.channel_conv(qkv, self.q_off, self.conv_w, cache.state.get(self.cache_key + ".conv"), step, out, first, self.v_off,
+                         self.mix_share, heads, first_heads)
+        if lead:
+            step.scratch[("attention.values", mix["group"])] = (out[:, self.v_off:self.v_off + self.KV * self.hd], heads)
+        return out
 
     def _joined(self, att: torch.Tensor, out: Optional[torch.Tensor]) -> torch.Tensor:
         """With two maps a head: the pairs' difference, normed (one kernel); else the kernels' result as it is."""

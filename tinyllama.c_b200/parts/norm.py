@@ -16,16 +16,20 @@ from .base import LayerCache, Part, StateRequest, StepInfo, WeightSpec, register
 
 @register_norm("rmsnorm")
 class RMSNorm(Part):
-    def __init__(self, width: int, eps: float, weight_name: str, offset: float = 0.0):
-        """offset: what is added to the stored weight (1.0 for a weight stored as its distance from one)."""
+    def __init__(self, width: int, eps: float, weight_name: str, offset: float = 0.0, one_gain: bool = False):
+        """offset: what is added to the stored weight (1.0 for a weight stored as its distance from one).  one_gain: the stored
+        weight is a single number for all coordinates (a tensor without dimensions)."""
         self.width, self.eps, self.weight_name, self.offset = int(width), float(eps), weight_name, float(offset)
+        self.one_gain = bool(one_gain)
         self.weight: Optional[torch.Tensor] = None
 
     def weight_specs(self) -> List[WeightSpec]:
-        return [WeightSpec(self.weight_name, (self.width,), "ones" if self.offset == 0.0 else "near_zero")]
+        return [WeightSpec(self.weight_name, () if self.one_gain else (self.width,), "ones" if self.offset == 0.0 else "near_zero")]
 
     def bind(self, tensors: Dict[str, torch.Tensor], dtype, device) -> None:
         self.weight = to_vec(tensors[self.weight_name], device)
+        if self.one_gain:
+            self.weight = self.weight.reshape(1).expand(self.width).contiguous()
         if self.offset != 0.0:
             self.weight = (self.weight + self.offset).contiguous()        # in 32 bits
 
@@ -98,6 +102,41 @@ class RMSNormShift(RMSNorm):
         if not cache.writes:
             raise ValueError("rmsnorm_shift: the kept row would advance twice in a step on another entry's cache")
         ops.rmsnorm_shift(x32, self.weight, self.mix, self.eps, cache.state[self.cache_key], step, out)
+        return out
+
+
+@register_norm("rmsnorm_conv")
+class RMSNormConv(RMSNorm):
+    """RMSNorm followed by a short causal convolution over time that is added to the normed row: with h[t] the normed row, the
+    result is h[t] + sum_j w[:, j] h[t - taps + 1 + j] (weights [D, taps], newest tap last, zeros before the sequence's first
+    row).  The last taps - 1 normed rows of a sequence are kept per sequence (32-bit) between steps; two such norms of one
+    layer need two cache keys."""
+
+    def __init__(self, width: int, eps: float, weight_name: str, conv_name: str, taps: int, one_gain: bool = False,
+                 cache_key: str = "norm_conv"):
+        super().__init__(width, eps, weight_name, one_gain=one_gain)
+        self.conv_name, self.taps, self.cache_key = conv_name, int(taps), cache_key
+        if not (1 <= self.taps <= ops.MAX_CONV_TAPS):
+            raise ValueError(f"rmsnorm_conv: {taps} convolution taps are outside what the kernels are built for (1..{ops.MAX_CONV_TAPS})")
+        self.conv_w: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> List[WeightSpec]:
+        return super().weight_specs() + [WeightSpec(self.conv_name, (self.width, self.taps), "conv")]
+
+    def cache_requests(self) -> list:
+        return [StateRequest(self.cache_key, (self.taps - 1, self.width))] if self.taps > 1 else []
+
+    def bind(self, tensors: Dict[str, torch.Tensor], dtype, device) -> None:
+        super().bind(tensors, dtype, device)
+        self.conv_w = to_vec(tensors[self.conv_name].t(), device)            # tap by tap
+
+    def forward(self, x32, out, rows=None):
+        raise ValueError("rmsnorm_conv: a norm with a convolution over time needs the step and the cache (forward_step)")
+
+    def forward_step(self, x32: torch.Tensor, out: torch.Tensor, step: StepInfo, cache: LayerCache) -> torch.Tensor:
+        if not cache.writes:
+            raise ValueError("rmsnorm_conv: the kept rows would advance twice in a step on another entry's cache")
+        ops.rmsnorm_conv(x32, self.weight, self.eps, self.conv_w, cache.state.get(self.cache_key), step, out)
         return out
 
 

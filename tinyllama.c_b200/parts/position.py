@@ -31,18 +31,19 @@ class RotaryNeox(Position):
         kind "ramp": with x(t) = r ln(original / (2 pi t)) / (2 ln theta) the (real) pair index whose wave makes t turns over
         `original` positions, lo = max(floor(x(fast)), 0), hi = min(ceil(x(slow)), r - 1) and ramp_i = clamp((i - lo) /
         max(hi - lo, 0.001), 0, 1): f_i / factor * ramp_i + f_i (1 - ramp_i), and every cosine and sine is multiplied by
-        0.1 ln(factor) + 1 (`amplitude`; a mixer that rotates by itself asks for it)."""
+        0.1 ln(factor) + 1 (`amplitude`; a mixer that rotates by itself asks for it).  kind "linear": every f_i / factor."""
         self.head_dim = int(head_dim)
         self.scaling = dict(scaling) if scaling else None
         self.amplitude = 1.0
         if self.scaling is not None:
             kind = self.scaling.get("kind")
-            need = {"bands": ("factor", "low", "high", "original"), "ramp": ("factor", "fast", "slow", "original")}.get(kind)
+            need = {"bands": ("factor", "low", "high", "original"), "ramp": ("factor", "fast", "slow", "original"),
+                    "linear": ("factor",)}.get(kind)
             if need is None or any(not isinstance(self.scaling.get(k), (int, float)) or isinstance(self.scaling.get(k), bool)
                                    for k in need):
-                raise ValueError(f"rotation scaling {scaling!r}: kind 'bands' (factor, low, high, original) or 'ramp' "
-                                 f"(factor, fast, slow, original), all numbers")
-            if self.scaling["factor"] <= 0 or self.scaling["original"] <= 0 or (kind == "bands" and self.scaling["high"] == self.scaling["low"]):
+                raise ValueError(f"rotation scaling {scaling!r}: kind 'bands' (factor, low, high, original), 'ramp' "
+                                 f"(factor, fast, slow, original) or 'linear' (factor), all numbers")
+            if self.scaling["factor"] <= 0 or self.scaling.get("original", 1) <= 0 or (kind == "bands" and self.scaling["high"] == self.scaling["low"]):
                 raise ValueError(f"rotation scaling {scaling!r}: factor and original must be positive, high and low differ")
         self.rope_dim = int(rope_dim) if rope_dim else self.head_dim      # falcon_h1.c:265
         if self.rope_dim % 2 or self.rope_dim > self.head_dim:
@@ -59,6 +60,8 @@ class RotaryNeox(Position):
             s = ((sc["original"] / wave - sc["low"]) / (sc["high"] - sc["low"]))
             blend = (1.0 - s) * inv / sc["factor"] + s * inv
             inv = torch.where(wave < sc["original"] / sc["high"], inv, torch.where(wave > sc["original"] / sc["low"], inv / sc["factor"], blend))
+        elif sc is not None and sc["kind"] == "linear":
+            inv = inv / sc["factor"]
         elif sc is not None:
             at = lambda turns: self.rope_dim * math.log(sc["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(self.theta))
             lo, hi = max(math.floor(at(sc["fast"])), 0), min(math.ceil(at(sc["slow"])), self.rope_dim - 1)
