@@ -245,9 +245,9 @@ def main() -> int:
     ap.add_argument("--no-big", dest="big", action="store_false", help="skip the 3B and 7B workloads among the points")
     ap.add_argument("--no-pairs", action="store_true", help="run the linear layers on single blocks (128 x 256 tiles) instead "
                     "of pairs of blocks on 256 x 256 tiles: the comparison behind profiles/linear_tcgen05_prefill_2048.md")
-    ap.add_argument("--design", default=None, choices=["turevik", "porarax", "sogazen", "kimutar"], help="instead of the benchmark line: prefill and decode "
+    ap.add_argument("--design", default=None, choices=["turevik", "porarax", "sogazen", "kimutar", "kefetar"], help="instead of the benchmark line: prefill and decode "
                     "throughput of this design at layer sizes of a real model's order (random weights), beside the library's "
-                    "closest other design (Falcon-H1 for turevik and sogazen, Turevik for porarax, Porarax for kimutar) at equal "
+                    "closest other design (Falcon-H1 for turevik and sogazen, Turevik for porarax, Porarax for kimutar, Kimutar for kefetar) at equal "
                     "width and layer count")
     ap.add_argument("--sizes-only", default=None, choices=["width 2048", "width 3072"], help="with --design: one of the two sizes")
     ap.add_argument("--ref-budget", type=float, default=600.0, help="seconds the reference arm may take (it runs fewer "
@@ -501,10 +501,10 @@ def kimutar_work(cfg, batch, context, T):
         m = layer["mixer"]
         H, G, dk, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
         if layer["type"] == "attention_2":
-            W = m["mask"]["size"]
+            seen = m["mask"]["size"] + m["mask"]["keep_first"] if "mask" in m else 1 << 30
             fixed += (H * dk + G * dk + G * dv) * D + D * H * dv
-            cache_bytes += batch * min(context, W + m["mask"]["keep_first"]) * G * (dk + dv) * 2
-            keys = sum(min(t + 1, W + m["mask"]["keep_first"]) for t in range(T)) if T > 1 else 1
+            cache_bytes += batch * min(context, seen) * G * (dk + dv) * 2
+            keys = sum(min(t + 1, seen) for t in range(T)) if T > 1 else 1
             mix_flops += 2.0 * H * (dk + dv) * keys
         elif layer["type"] == "attention":
             fixed += (2 * H * dk + 2 * G * dk + G * dv) * D + D * H * dv
@@ -528,9 +528,53 @@ def kimutar_work(cfg, batch, context, T):
     return (fixed - V * D) * 2 + expert_bytes + cache_bytes, 2.0 * (fixed - 2 * V * D + expert_params) * T + 2.0 * V * D + mix_flops
 
 
+def kefetar_config(width, heads, kv_heads, ff, vocab):
+    """Four layers with every kind of mixer, a dense feed-forward in each: retention; attention with convolved q, k and v, capped
+    scores and an output gate, whose values lead the blended ones; retention; attention with blended values."""
+    decay = [1.0 - 2.0 ** (-5.0 - 5.0 * h / heads) for h in range(heads)]
+    ret = dict(type="retention", mixer=dict(heads=heads, dim=128, vdim=128, decay=decay, rot=dict(base=10000.0, dims=128)),
+               mlp=dict(kind="dense", ff=ff))
+    att = dict(type="attention", mixer=dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, conv=4, scale=128 ** -0.5, softcap=50.0, v_mix=True,
+                                            rot=dict(base=500000.0, dims=128, scaling=dict(factor=8.0))), mlp=dict(kind="dense", ff=ff))
+    return dict(architecture="Kefetar", vocab=vocab, width=width, norm=dict(eps=1e-6), canon=dict(taps=4), layers=[ret, att, ret, att])
+
+
+def kimutar_dense_config(width, heads, kv_heads, ff, vocab):
+    """Kimutar's layers that are nearest to Kefetar's, at the same sizes and in the same order: the delta rule with a decay per
+    channel, attention without a window, a dense feed-forward in each."""
+    delta = dict(type="channel_delta", mixer=dict(heads=heads, kv_heads=heads, dim=128, vdim=128, conv=4, decay_rank=width // 16,
+                                                  gate_rank=width // 16), mlp=dict(kind="dense", ff=ff))
+    att = dict(type="attention_2", mixer=dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5,
+                                              rot=dict(base=500000.0, dims=128, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))),
+               mlp=dict(kind="dense", ff=ff))
+    return dict(architecture="Kimutar", vocab=vocab, width=width, norm=dict(eps=1e-6), layers=[delta, att, delta, att])
+
+
+def kefetar_work(cfg, batch, context, T):
+    """(bytes a decode step of `batch` sequences at `context` must read, FLOPs of a prompt of T tokens)."""
+    D, V, taps = cfg["width"], cfg["vocab"], cfg["canon"]["taps"]
+    fixed, cache_bytes, mix_flops = V * D, 0, 0.0                         # the head (the table is read by rows)
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        H, dk, dv = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "retention":
+            fixed += (2 * H * dk + 2 * H * dv) * D + D * H * dv
+            cache_bytes += batch * H * dk * dv * 4                        # the state, 32-bit
+            mix_flops += 4.0 * H * dk * dv * T                            # the write k v^T and the read-out S^T q
+        else:
+            G = m["kv_heads"]
+            fixed += (H * dk + G * dk + G * dv + H * dv) * D + D * H * dv
+            cache_bytes += batch * context * G * (dk + dv) * 2 + batch * (m["conv"] - 1) * (H * dk + G * (dk + dv)) * 4
+            mix_flops += 2.0 * H * (dk + dv) * T * (T + 1) / 2
+        cache_bytes += batch * (taps - 1) * D * 4 * (2 if layer["mlp"] else 1)
+        if layer["mlp"]:
+            fixed += 2 * D * layer["mlp"]["ff"]
+    return fixed * 2 + cache_bytes, 2.0 * (fixed - V * D) * T + 2.0 * V * D + mix_flops
+
+
 def design_compare(args) -> int:
     """Another design beside the library's closest one at equal width and layer count (Turevik and Sogazen beside Falcon-H1,
-    Porarax beside Turevik, Kimutar beside Porarax): a prompt of --prefill-tokens tokens and decode steps at batch 8 and 64 from --prompt-len-token
+    Porarax beside Turevik, Kimutar beside Porarax, Kefetar beside Kimutar): a prompt of --prefill-tokens tokens and decode steps at batch 8 and 64 from --prompt-len-token
     prompts, each as time and as a fraction of the measured peak for the bytes a step must read (decode) or the FLOPs a
     prompt needs (prefill)."""
     import torch
@@ -549,6 +593,10 @@ def design_compare(args) -> int:
         cases = {"width 2048": (kimutar_config(2048, 16, 4, 1024, 4096, 32, 4, 1024, 1024, 65536), porarax["width 2048"]),
                  "width 3072": (kimutar_config(3072, 24, 8, 1024, 12288, 64, 6, 2048, 2048, 130048), porarax["width 3072"])}
         beside = "porarax"
+    elif args.design == "kefetar":
+        sizes_of = {"width 2048": (2048, 16, 4, 4096, 65536), "width 3072": (3072, 24, 8, 12288, 130048)}
+        cases = {k: (kefetar_config(*v), kimutar_dense_config(*v)) for k, v in sizes_of.items()}
+        beside = "kimutar"
     elif args.design == "sogazen":
         cases = {"width 2048": (sogazen_config(2048, 8, 2, 48, 64, 256, 32, 4096, 32, 4, 4, 1024, 65536), dict(CONFIG_1P5B, num_hidden_layers=4)),
                  "width 3072": (sogazen_config(3072, 12, 2, 24, 128, 256, 48, 12288, 64, 8, 6, 2048, 130048), dict(CONFIG_7B, num_hidden_layers=4))}
@@ -557,7 +605,8 @@ def design_compare(args) -> int:
         cases = {"width 2048": (turevik["width 2048"], dict(CONFIG_1P5B, num_hidden_layers=4)),
                  "width 3072": (turevik["width 3072"], dict(CONFIG_7B, num_hidden_layers=4))}
         beside = "falcon_h1"
-    work = {"turevik": turevik_work, "porarax": porarax_work, "sogazen": sogazen_work, "kimutar": kimutar_work}
+    work = {"turevik": turevik_work, "porarax": porarax_work, "sogazen": sogazen_work, "kimutar": kimutar_work,
+            "kefetar": kefetar_work}
     if args.sizes_only:
         cases = {k: v for k, v in cases.items() if k == args.sizes_only}
     for name, (tcfg, fcfg) in cases.items():

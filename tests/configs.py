@@ -347,3 +347,75 @@ def kimutar_random(seed: int) -> dict:
         start = int(rng.integers(0, len(layers)))
         cfg["loop"] = dict(start=start, stop=int(rng.integers(start + 1, len(layers) + 1)), times=pick(1, 2, 3))
     return cfg
+
+
+# ---- Kefetar ------------------------------------------------------------------------------------------------------------------
+def _kef_rot(base, dims, factor=None):
+    rot = dict(base=base, dims=dims)
+    if factor:
+        rot["scaling"] = dict(factor=factor)
+    return rot
+
+
+def _kef_ret(heads, dim, vdim, decay, rot, ff):
+    return dict(type="retention", mixer=dict(heads=heads, dim=dim, vdim=vdim, decay=list(decay), rot=rot), mlp=_k_dense(ff) if ff else None)
+
+
+def _kef_att(heads, kv_heads, dim, vdim, conv, scale, softcap, v_mix, rot, ff):
+    m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, conv=conv, scale=scale, v_mix=v_mix, rot=rot)
+    if softcap:
+        m["softcap"] = softcap
+    return dict(type="attention", mixer=m, mlp=_k_dense(ff) if ff else None)
+
+
+# A: attention first, without a share in the blended values; a width and a feed-forward that are no multiples of 8; three
+# taps in front of every sublayer; retention heads of 12 x 20 (values wider than keys, a third of the keys rotated) and of
+# 10 x 6 (no multiple of 4, without rotation, a decay of one and a fast one); blended values in three layers whose heads lie
+# differently (2 x 16 behind keys of 24, 1 x 32 behind keys of 20, 4 x 8 behind keys of 8), one, two and four taps on q, k
+# and v; scores with and without a cap; frequencies divided and plain; layers without feed-forward; six query heads a key head
+KEFETAR_A = dict(architecture="Kefetar", vocab=150, width=52, norm=dict(eps=1e-5), canon=dict(taps=3), layers=[
+    _kef_att(4, 2, 24, 16, 2, 0.3, 4.0, False, _kef_rot(100.0, 8, 3.0), 44),
+    _kef_ret(3, 12, 20, [0.9, 0.97, 0.995], _kef_rot(1000.0, 4), None),
+    _kef_att(2, 2, 24, 16, 4, 0.25, None, True, _kef_rot(10000.0, 24), 36),
+    _kef_att(6, 1, 20, 32, 1, 0.2, 6.0, True, _kef_rot(500.0, 6, 2.5), None),
+    _kef_ret(2, 10, 6, [1.0, 0.5], _kef_rot(100.0, 0), 20),
+    _kef_att(4, 4, 8, 8, 3, 0.4, 3.0, True, _kef_rot(3000.0, 8), 28),
+])
+
+# B: heads of 64 and of 128 (the tcgen05 attention of prompts, the one-kernel attention of single tokens), retention heads of
+# 64 x 64 and of 32 x 48 (the chunked form on the tensor cores), five taps in front of every sublayer, retention first
+KEFETAR_B = dict(architecture="Kefetar", vocab=97, width=64, norm=dict(eps=1e-6), canon=dict(taps=5), layers=[
+    _kef_ret(2, 64, 64, [0.98, 0.9995], _kef_rot(50000.0, 64), 80),
+    _kef_att(4, 2, 64, 64, 3, 0.11, 9.0, True, _kef_rot(20000.0, 32, 4.0), 96),
+    _kef_ret(3, 32, 48, [0.93, 0.99, 0.999], _kef_rot(700.0, 16), None),
+    _kef_att(2, 1, 128, 128, 2, 0.07, 12.0, True, _kef_rot(1000000.0, 128, 8.0), 40),
+    _kef_att(2, 2, 64, 40, 4, 0.12, None, False, _kef_rot(300.0, 16), 64),
+])
+
+KEFETAR = {"FA": KEFETAR_A, "FB": KEFETAR_B}
+
+
+def kefetar_random(seed: int) -> dict:
+    """A Kefetar configuration drawn from `seed`: 2 to 6 layers of both kinds in any order, with head counts, sizes, rotated
+    dimensions, scalings, taps, caps, decays, feed-forwards and constants all drawn (blended values have one size per model)."""
+    import numpy as np
+    rng = np.random.default_rng(seed)
+    pick = lambda *v: v[int(rng.integers(len(v)))]
+    layers, values = [], pick(16, 32, 48, 64)
+    for _ in range(int(rng.integers(2, 7))):
+        ff = pick(None, 8, 20, 36, 64)
+        dim = pick(8, 10, 16, 24, 32, 64, 128)
+        dims = pick(0, 2, dim // 4 * 2, dim)
+        base = pick(50.0, 10000.0, 500000.0)
+        if rng.random() < 0.5:
+            heads = pick(1, 2, 3, 5)
+            decay = [float(pick(0.5, 0.9, 0.97, 0.99, 0.999, 1.0)) for _ in range(heads)]
+            layers.append(_kef_ret(heads, dim, pick(6, 8, 16, 20, 32, 64), decay, _kef_rot(base, dims), ff))
+            continue
+        v_mix = bool(rng.random() < 0.6)
+        kv = pick(1, 2, 4)
+        vdim = values // kv if v_mix else pick(6, 8, 20, 32, 64)
+        layers.append(_kef_att(kv * pick(1, 2, 3, 5), kv, dim, vdim, pick(1, 2, 3, 4, 6), float(dim ** -0.5 * rng.uniform(0.5, 2.0)),
+                               pick(None, 2.0, 10.0), v_mix, _kef_rot(base, dims, pick(None, 1.5, 4.0)), ff))
+    return dict(architecture="Kefetar", vocab=pick(50, 131, 300), width=pick(32, 44, 50, 64, 96), norm=dict(eps=pick(1e-5, 1e-6)),
+                canon=dict(taps=pick(1, 2, 3, 4, 6)), layers=layers)

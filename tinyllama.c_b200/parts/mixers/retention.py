@@ -73,26 +73,30 @@ class RetentionMixer(Part):
         self._one = torch.ones(self.H * self.dv, dtype=torch.float32, device=device)
 
     def forward(self, normed: torch.Tensor, step: StepInfo, cache: LayerCache, residual: torch.Tensor, accumulate: bool = True) -> None:
+        proj = scratch_buf(f"retention.{self.cache_key}.proj", (step.n_rows, self.proj.out_features), torch.float32, normed.device)
+        self.proj.forward(normed, proj)
+        self.o.forward(self.mix(proj, step, cache), residual, accumulate=accumulate)
+
+    def mix(self, proj: torch.Tensor, step: StepInfo, cache: LayerCache) -> torch.Tensor:
+        """Everything between the projections (float32 [T, q | k | v | g]) and the output projection: [T, H * dv]."""
         if not cache.writes:
             raise ValueError("retention: a recurrent mixer cannot run on another layer's cache without storing "
                              "(its state would advance twice in one step)")
-        T, dev, f32 = step.n_rows, normed.device, torch.float32
+        T, dev, f32 = step.n_rows, proj.device, torch.float32
         new = lambda tag, shape, dt: scratch_buf(f"retention.{self.cache_key}.{tag}", shape, dt, dev)
         H, dk, dv = self.H, self.dk, self.dv
-        proj = new("proj", (T, self.proj.out_features), f32)
-        self.proj.forward(normed, proj)
         gated = new("gated", (T, H * dv), self.dtype)
         state, table = cache.state[self.cache_key], self.position.rotation_table()
         if step.max_new == 1:
             ops.retention_decode(proj, self.q_off, self.k_off, self.v_off, self.g_off, table, self.decays, self.k_scale, self.eps, state,
                                  step, H, dk, dv, gated)
-        else:
-            vkq = new("vkq", (T, H * (dv + 2 * dk)), f32)
-            ones, decays = new("ones", (T, H), f32), new("decays", (T, H), f32)
-            ops.retention_prepare(proj, self.q_off, self.k_off, self.v_off, table, step.positions, self.decays, self.k_scale, H, dk, dv,
-                                  vkq, ones, decays)
-            y = new("y", (T, H * dv), f32)
-            ops.ssm_scan(vkq, ones, decays, self._no_skip, state, step.cu_seqlens, step.slots, step.start_pos, y, H, dv, dk, H,
-                         step.chunks.get(self.scan_chunk))
-            ops.gated_rmsnorm(y, proj[:, self.g_off:self.g_off + H * dv], self._one, self.eps, H, True, gated)
-        self.o.forward(gated, residual, accumulate=accumulate)
+            return gated
+        vkq = new("vkq", (T, H * (dv + 2 * dk)), f32)
+        ones, decays = new("ones", (T, H), f32), new("decays", (T, H), f32)
+        ops.retention_prepare(proj, self.q_off, self.k_off, self.v_off, table, step.positions, self.decays, self.k_scale, H, dk, dv,
+                              vkq, ones, decays)
+        y = new("y", (T, H * dv), f32)
+        ops.ssm_scan(vkq, ones, decays, self._no_skip, state, step.cu_seqlens, step.slots, step.start_pos, y, H, dv, dk, H,
+                     step.chunks.get(self.scan_chunk))
+        ops.gated_rmsnorm(y, proj[:, self.g_off:self.g_off + H * dv], self._one, self.eps, H, True, gated)
+        return gated
