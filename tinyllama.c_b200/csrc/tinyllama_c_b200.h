@@ -432,6 +432,16 @@ int tlc_retention_prepare(const float* proj, int ld, int q_off, int k_off, int v
 int tlc_retention_decode(const float* proj, int ld, int q_off, int k_off, int v_off, int g_off, const float* inv_freq, int rope_dim,
                          const int* positions, const int* slots, const float* decay, float k_scale, float eps, float* state, int B,
                          int H, int dk, int dv, void* out, int out_dtype, int out_ld, cudaStream_t stream);
+/* Prompts in chunks of at most 64 rows (sizes of tlc_retention_chunks_ok): the same result as prepare + scan + norm + gate with
+ * every product of 32-bit values formed from pairs of TF32 numbers on the tensor cores.  q and k are rotated in place in proj;
+ * scratch: n_seg * H * (dk * dv + 1) floats; chunk tables as for tlc_ssm_scan_chunked. */
+int tlc_retention_init(void);
+int tlc_retention_chunks_ok(int dk, int dv, int rope_dim);
+int tlc_retention_chunked(float* proj, int ld, int q_off, int k_off, int v_off, int g_off, const float* inv_freq, int rope_dim,
+                          const int* positions, const float* decay, float k_scale, float eps, float* state, float* scratch,
+                          const int* seg_start, const int* seg_seq, const int* seq_seg_start, const int* slots, const int* start_pos,
+                          int B, int n_seg, int chunk_rows, int H, int dk, int dv, void* out, int out_dtype, int out_ld,
+                          cudaStream_t stream);
 
 /* ---- sampling (sampling.cu) ------------------------------------------------------------------------ */
 /* out[r] = first index of the maximum of logits[r].  work: NULL (one block a row), or 12 * R bytes, 8-byte

@@ -106,6 +106,10 @@ _SIGNATURES = {
     "tlc_polynorm": (_i, [_vp, _i, _i, _i, _f, _f, _f, _f, _f, _vp, _i, _vp]),
     "tlc_retention_prepare": (_i, [_vp, _i, _i, _i, _i, _vp, _i, _vp, _vp, _f, _i, _i, _i, _i, _vp, _vp, _vp, _vp]),
     "tlc_retention_decode": (_i, [_vp, _i, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _f, _f, _vp, _i, _i, _i, _i, _vp, _i, _i, _vp]),
+    "tlc_retention_init": (_i, []),
+    "tlc_retention_chunks_ok": (_i, [_i, _i, _i]),
+    "tlc_retention_chunked": (_i, [_vp, _i, _i, _i, _i, _i, _vp, _i, _vp, _vp, _f, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i,
+                                   _i, _i, _vp, _i, _i, _vp]),
     "tlc_moe_identity": (_i, [_vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _vp, _vp]),
     "tlc_rmsnorm_shift": (_i, [_vp, _vp, _vp, _f, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp]),
     "tlc_rmsnorm_add": (_i, [_vp, _i, _vp, _vp, _i, _i, _vp, _f, _i, _i, _vp, _i, _vp, _i, _vp]),
@@ -153,7 +157,7 @@ def library() -> ctypes.CDLL:
             fn.restype = restype
         _lib = lib
         if torch.cuda.is_available():                                     # before any stream capture
-            for init in (lib.tlc_linear_init, lib.tlc_attention_prefill_init, lib.tlc_ssd_init):
+            for init in (lib.tlc_linear_init, lib.tlc_attention_prefill_init, lib.tlc_ssd_init, lib.tlc_retention_init):
                 if init() != 0:
                     raise KernelError(f"kernel library set-up: {lib.tlc_last_error().decode()}")
         # Programmatic dependent launch for every kernel of the library, captured or not: a kernel's blocks are
@@ -1462,4 +1466,41 @@ def retention_decode(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_o
     _call("tlc_retention_decode", proj.data_ptr(), ld, int(q_off), int(k_off), int(v_off), int(g_off), inv_freq.data_ptr(),
           2 * inv_freq.numel(), step.positions.data_ptr(), step.slots.data_ptr(), decay.data_ptr(), float(k_scale), float(eps),
           state.data_ptr(), B, int(H), int(dk), int(dv), out.data_ptr(), dtype_code(out.dtype), _out_rows(out, B, H * dv, "retention_decode"),
+          _stream())
+
+
+RETENTION_CHUNK = 64             # retention.cu: rows of a chunk of prompts on the tensor cores (at most)
+_retention_chunks = not bool(int(os.environ.get("TLC_DISABLE_RETENTION_CHUNKS", "0")))
+
+
+def retention_chunks(on: bool) -> None:
+    """Whether prompts of a bfloat16 run take the chunk kernels where they are built (TLC_DISABLE_RETENTION_CHUNKS=1 sets the
+    start value to off); for tests and comparisons."""
+    global _retention_chunks
+    _retention_chunks = bool(on)
+
+
+def retention_chunked_ok(proj: torch.Tensor, offsets, dk: int, dv: int, rope_dim: int, chunk_rows: int) -> bool:
+    return bool(_retention_chunks and chunk_rows <= RETENTION_CHUNK and library().tlc_retention_chunks_ok(dk, dv, rope_dim)
+                and _rows(proj, "retention projection") % 4 == 0 and proj.data_ptr() % 16 == 0 and all(o % 4 == 0 for o in offsets))
+
+
+def retention_chunked(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, inv_freq: torch.Tensor, decay: torch.Tensor,
+                      k_scale: float, eps: float, state: torch.Tensor, step, chunks, chunk_rows: int, H: int, dk: int, dv: int,
+                      out: torch.Tensor) -> None:
+    """Prompts: what retention_decode computes, for every row of the step, in chunks that run side by side (chunks: the step's
+    chunk table for chunk_rows); the products of 32-bit values run on the tensor cores, each operand as a pair of TF32
+    numbers.  proj's q and k columns are rotated in place.  See retention_chunked_ok for what it takes."""
+    ld = _retention_checks(proj, inv_freq, decay, state, H, dk, dv, ((q_off, H * dk), (k_off, H * dk), (v_off, H * dv), (g_off, H * dv)),
+                           "retention_chunked")
+    seg_start, seg_seq, seq_seg_start = chunks
+    _gpu(out, seg_start, seg_seq, seq_seg_start)
+    n_seg, T = seg_seq.numel(), proj.shape[0]
+    scratch = torch.empty(n_seg * H * (dk * dv + 1), dtype=torch.float32, device=proj.device)
+    global _launches
+    _launches += 2                      # (three kernels)
+    _call("tlc_retention_chunked", proj.data_ptr(), ld, int(q_off), int(k_off), int(v_off), int(g_off), inv_freq.data_ptr(),
+          2 * inv_freq.numel(), step.positions.data_ptr(), decay.data_ptr(), float(k_scale), float(eps), state.data_ptr(), scratch.data_ptr(),
+          seg_start.data_ptr(), seg_seq.data_ptr(), seq_seg_start.data_ptr(), step.slots.data_ptr(), step.start_pos.data_ptr(), step.n_seqs,
+          n_seg, int(chunk_rows), int(H), int(dk), int(dv), out.data_ptr(), dtype_code(out.dtype), _out_rows(out, T, H * dv, "retention_chunked"),
           _stream())

@@ -9,8 +9,10 @@ dk ** -0.5.  Per head, with the head's decay a (a constant of the layer) and the
 and W_o maps the heads' results back.  S is kept per sequence between steps, 32-bit, value by value ([H, dv, dk]);
 everything between the projections and the output projection is 32-bit.
 
-One-token steps run one kernel between the two products.  Prompts run the selective scan's kernels: with a step size of
-one, the decay as a step's factor and k and q as its input and output vectors that recurrence is this one.
+One-token steps run one kernel between the two products.  Prompts of a bfloat16 run are cut into chunks whose products run
+on the tensor cores, every 32-bit operand as a pair of TF32 numbers.  Everything else (32-bit runs, short portions, head
+sizes the chunk kernels are not built for) runs the selective scan's 32-bit kernels: with a step size of one, the decay as a
+step's factor and k and q as its input and output vectors that recurrence is this one.
 """
 from __future__ import annotations
 
@@ -26,7 +28,7 @@ from ..linear import StackedLinear
 @register_mixer("retention")
 class RetentionMixer(Part):
     def __init__(self, hidden: int, n_heads: int, key_dim: int, v_dim: int, decay: Sequence[float], eps: float, position: PartSpec,
-                 names: Dict[str, str], cache_key: str = "retention", scan_chunk: int = 64):
+                 names: Dict[str, str], cache_key: str = "retention", scan_chunk: int = ops.RETENTION_CHUNK):
         """decay: one number per head.  eps: of the heads' norm.  names: tensor names of q, k, v, g, o.  scan_chunk: rows of a
         chunk of the parallel scan of prompts (the result does not depend on it: the state is linear in its initial value)."""
         self.hidden, self.H, self.dk, self.dv = int(hidden), int(n_heads), int(key_dim), int(v_dim)
@@ -90,6 +92,12 @@ class RetentionMixer(Part):
         if step.max_new == 1:
             ops.retention_decode(proj, self.q_off, self.k_off, self.v_off, self.g_off, table, self.decays, self.k_scale, self.eps, state,
                                  step, H, dk, dv, gated)
+            return gated
+        chunks = step.chunks.get(self.scan_chunk)
+        if self.dtype == torch.bfloat16 and chunks is not None and ops.retention_chunked_ok(
+                proj, (self.q_off, self.k_off, self.v_off, self.g_off), dk, dv, 2 * table.numel(), self.scan_chunk):
+            ops.retention_chunked(proj, self.q_off, self.k_off, self.v_off, self.g_off, table, self.decays, self.k_scale, self.eps, state,
+                                  step, chunks, self.scan_chunk, H, dk, dv, gated)
             return gated
         vkq = new("vkq", (T, H * (dv + 2 * dk)), f32)
         ones, decays = new("ones", (T, H), f32), new("decays", (T, H), f32)
