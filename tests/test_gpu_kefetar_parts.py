@@ -209,6 +209,37 @@ def test_retention(dtype, H, dk, dv, rot):
         assert np.abs(got[i] - want).max() <= tol * np.abs(want).max(), f"short sequence {i}"
 
 
+@pytest.mark.parametrize("H,dk,dv,rot", [(3, 128, 128, 128), (2, 64, 96, 32), (2, 36, 72, 8), (4, 32, 32, 0), (1, 100, 128, 96), (2, 8, 4, 8)])
+def test_retention_in_chunks_to_32_bits(H, dk, dv, rot):
+    """The chunk kernels with a 32-bit result: pairs of TF32 numbers must give what 32-bit products give.  Two prompts of many
+    chunks, one of which goes on (its state and an odd last chunk), a third of a single row."""
+    g = np.random.default_rng(dk)
+    decay, eps = [0.9995, 1.0, 0.7, 0.98][:H], 1e-5
+    freq = plain.frequencies(dict(base=3000.0, dims=rot)) if rot else np.zeros(0)
+    state = torch.full((4, H, dv, dk), 5.0, device="cuda")
+    width = 2 * H * (dk + dv) + 8
+    offs = [4, 4 + H * dk, 4 + 2 * H * dk, 4 + 2 * H * dk + H * dv]
+    seqs = [g.standard_normal((n, width)).astype(np.float32).astype(np.float64) for n in (211, 150, 2)]
+
+    def call(rows, step):
+        assert ops.retention_chunked_ok(dev(rows), offs, dk, dv, rot, 64)
+        out = torch.empty((len(rows), H * dv), device="cuda")
+        ops.retention_chunked(dev(rows), *offs, dev(freq), dev(decay), dk ** -0.5, eps, state, step, step.chunks[64], 64, H, dk, dv, out)
+        torch.cuda.synchronize()
+        return out.cpu().numpy().astype(np.float64)
+
+    got = run_schedule(seqs, [0, 3, 1], [[130, 81], [65, 85], [1, 1]], call, chunk_rows=64, chunk_from=0)
+    for i, s in enumerate(seqs):
+        T = len(s)
+        take = lambda o, n: s[:, o:o + H * n].reshape(T, H, n)
+        q = plain.rotate_halves(take(offs[0], dk), np.arange(T), freq)
+        k = plain.rotate_halves(take(offs[1], dk), np.arange(T), freq) * dk ** -0.5
+        o = np.stack([plain.retention_scan(q[:, h], k[:, h], take(offs[2], dv)[:, h], decay[h]) for h in range(H)], axis=1)
+        want = plain.unit_rms(o, eps).reshape(T, -1) * plain.silu(s[:, offs[3]:offs[3] + H * dv])
+        err = np.abs(got[i] - want).max(1)
+        assert err.max() <= 3e-5 * np.abs(want).max(), f"sequence {i} row {int(err.argmax())}: {err.max():.3e} of {np.abs(want).max():.3e}"
+
+
 # ---- capped scores without a sink ---------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", list(DT))
 @pytest.mark.parametrize("H,KV,hd", [(6, 3, 24), (4, 2, 64), (4, 1, 80), (8, 2, 128)])

@@ -215,10 +215,24 @@ struct TileA {
     lo[0] = s0.lo; lo[1] = s1.lo; lo[2] = s2.lo; lo[3] = s3.lo;
   }
 };
-__device__ __forceinline__ void mma_split(float (&c)[4], const TileA& a, const Split& b0, const Split& b1) {
-  mma_tf32(c, a.lo, b0.hi, b1.hi);
-  mma_tf32(c, a.hi, b0.lo, b1.lo);
-  mma_tf32(c, a.hi, b0.hi, b1.hi);
+// The three products of M x Q tiles, one kind after the other, so that products into one accumulator do not follow one another.
+template <int M, int Q, int N>
+__device__ __forceinline__ void mma_split(float (&c)[M][N][4], int q0, const TileA (&a)[M], const Split (&b)[Q][2]) {
+#pragma unroll
+  for (int q = 0; q < Q; q++)
+#pragma unroll
+    for (int m = 0; m < M; m++)
+      if (q0 + q < N) mma_tf32(c[m][q0 + q < N ? q0 + q : 0], a[m].lo, b[q][0].hi, b[q][1].hi);
+#pragma unroll
+  for (int q = 0; q < Q; q++)
+#pragma unroll
+    for (int m = 0; m < M; m++)
+      if (q0 + q < N) mma_tf32(c[m][q0 + q < N ? q0 + q : 0], a[m].hi, b[q][0].lo, b[q][1].lo);
+#pragma unroll
+  for (int q = 0; q < Q; q++)
+#pragma unroll
+    for (int m = 0; m < M; m++)
+      if (q0 + q < N) mma_tf32(c[m][q0 + q < N ? q0 + q : 0], a[m].hi, b[q][0].hi, b[q][1].hi);
 }
 
 __device__ __forceinline__ void ret_cp16(float* dst, const float* src) {
@@ -246,12 +260,35 @@ retention_chunk_state_kernel(float* proj, int ld, int q_off, int k_off, int v_of
   const int t0 = seg_start[seg], n = min(seg_start[seg + 1] - t0, RET_C);
   const float a = decay[h];
   if (tid <= RET_C) pw[tid] = powf(a, (float)tid);
+  if (n < RET_C || dk < DKP || dv < DVP)                  // rows and columns that no copy fills
+    for (int i = tid; i < RET_C * (LDK + LDV); i += 256) sh[i] = 0.f;
+  // pairs of four dimensions each (the rotated ones), then four dimensions that are only scaled; a thread takes BATCH items
+  // at a time and fetches the first ones before the cosines are computed
+  constexpr int BATCH = 4;
+  const int p4 = half >> 2, per = p4 + ((dk - 2 * half) >> 2), items = n * per;
+  float4 qa[BATCH], qb[BATCH], ka[BATCH], kb[BATCH];
+  auto fetch = [&](int i0) {
+#pragma unroll
+    for (int u = 0; u < BATCH; u++) {
+      const int i = i0 + 256 * u;
+      if (i >= items) break;
+      const int r = i / per, it = i - r * per;
+      const float* row = proj + (size_t)(t0 + r) * ld + (size_t)h * dk;
+      if (it < p4) {
+        qa[u] = *reinterpret_cast<const float4*>(row + q_off + 4 * it);
+        qb[u] = *reinterpret_cast<const float4*>(row + q_off + half + 4 * it);
+        ka[u] = *reinterpret_cast<const float4*>(row + k_off + 4 * it);
+        kb[u] = *reinterpret_cast<const float4*>(row + k_off + half + 4 * it);
+      } else {
+        ka[u] = *reinterpret_cast<const float4*>(row + k_off + 2 * half + 4 * (it - p4));
+      }
+    }
+  };
+  fetch(tid);
   for (int i = tid; i < n * half; i += 256) {
     const int r = i / half, j = i - r * half;
     sincosf((float)positions[t0 + r] * inv_freq[j], &cs[r * 2 * half + half + j], &cs[r * 2 * half + j]);
   }
-  if (n < RET_C || dk < DKP || dv < DVP)                  // rows and columns that no copy fills
-    for (int i = tid; i < RET_C * (LDK + LDV); i += 256) sh[i] = 0.f;
   __syncthreads();
   const int dv4 = dv >> 2;
   for (int i = tid; i < n * dv4; i += 256) {
@@ -259,36 +296,38 @@ retention_chunk_state_kernel(float* proj, int ld, int q_off, int k_off, int v_of
     ret_cp16(vs + r * LDV + c, proj + (size_t)(t0 + r) * ld + v_off + (size_t)h * dv + c);
   }
   ret_cp_commit();
-  // pairs of four dimensions each (the rotated ones), then four dimensions that are only scaled
-  const int p4 = half >> 2, per = p4 + ((dk - 2 * half) >> 2);
-  for (int i = tid; i < n * per; i += 256) {
-    const int r = i / per, it = i - r * per;
-    float* qr = proj + (size_t)(t0 + r) * ld + q_off + (size_t)h * dk;
-    float* kr = proj + (size_t)(t0 + r) * ld + k_off + (size_t)h * dk;
-    const float w = pw[n - 1 - r];
-    float* kd = ks + r * LDK;
-    if (it < p4) {
-      const int d = 4 * it;
-      const float4 c = *reinterpret_cast<const float4*>(cs + r * 2 * half + d), s = *reinterpret_cast<const float4*>(cs + r * 2 * half + half + d);
-      float4 u = *reinterpret_cast<float4*>(qr + d), x = *reinterpret_cast<float4*>(qr + half + d);
-      *reinterpret_cast<float4*>(qr + d) = make_float4(u.x * c.x - x.x * s.x, u.y * c.y - x.y * s.y, u.z * c.z - x.z * s.z, u.w * c.w - x.w * s.w);
-      *reinterpret_cast<float4*>(qr + half + d) = make_float4(x.x * c.x + u.x * s.x, x.y * c.y + u.y * s.y, x.z * c.z + u.z * s.z, x.w * c.w + u.w * s.w);
-      u = *reinterpret_cast<float4*>(kr + d);
-      x = *reinterpret_cast<float4*>(kr + half + d);
-      const float4 lo = make_float4((u.x * c.x - x.x * s.x) * k_scale, (u.y * c.y - x.y * s.y) * k_scale, (u.z * c.z - x.z * s.z) * k_scale,
-                                    (u.w * c.w - x.w * s.w) * k_scale);
-      const float4 hi = make_float4((x.x * c.x + u.x * s.x) * k_scale, (x.y * c.y + u.y * s.y) * k_scale, (x.z * c.z + u.z * s.z) * k_scale,
-                                    (x.w * c.w + u.w * s.w) * k_scale);
-      *reinterpret_cast<float4*>(kr + d) = lo;
-      *reinterpret_cast<float4*>(kr + half + d) = hi;
-      *reinterpret_cast<float4*>(kd + d) = make_float4(lo.x * w, lo.y * w, lo.z * w, lo.w * w);
-      *reinterpret_cast<float4*>(kd + half + d) = make_float4(hi.x * w, hi.y * w, hi.z * w, hi.w * w);
-    } else {
-      const int d = 2 * half + 4 * (it - p4);
-      float4 u = *reinterpret_cast<float4*>(kr + d);
-      u = make_float4(u.x * k_scale, u.y * k_scale, u.z * k_scale, u.w * k_scale);
-      *reinterpret_cast<float4*>(kr + d) = u;
-      *reinterpret_cast<float4*>(kd + d) = make_float4(u.x * w, u.y * w, u.z * w, u.w * w);
+  for (int i0 = tid; i0 < items; i0 += 256 * BATCH) {
+    if (i0 != tid) fetch(i0);
+#pragma unroll
+    for (int u = 0; u < BATCH; u++) {
+      const int i = i0 + 256 * u;
+      if (i >= items) break;
+      const int r = i / per, it = i - r * per;
+      float* row = proj + (size_t)(t0 + r) * ld + (size_t)h * dk;
+      const float w = pw[n - 1 - r];
+      float* kd = ks + r * LDK;
+      if (it < p4) {
+        const int d = 4 * it;
+        const float4 c = *reinterpret_cast<const float4*>(cs + r * 2 * half + d), s = *reinterpret_cast<const float4*>(cs + r * 2 * half + half + d);
+        float4 y = qa[u], x = qb[u];
+        *reinterpret_cast<float4*>(row + q_off + d) = make_float4(y.x * c.x - x.x * s.x, y.y * c.y - x.y * s.y, y.z * c.z - x.z * s.z, y.w * c.w - x.w * s.w);
+        *reinterpret_cast<float4*>(row + q_off + half + d) = make_float4(x.x * c.x + y.x * s.x, x.y * c.y + y.y * s.y, x.z * c.z + y.z * s.z, x.w * c.w + y.w * s.w);
+        y = ka[u];
+        x = kb[u];
+        const float4 lo = make_float4((y.x * c.x - x.x * s.x) * k_scale, (y.y * c.y - x.y * s.y) * k_scale, (y.z * c.z - x.z * s.z) * k_scale,
+                                      (y.w * c.w - x.w * s.w) * k_scale);
+        const float4 hi = make_float4((x.x * c.x + y.x * s.x) * k_scale, (x.y * c.y + y.y * s.y) * k_scale, (x.z * c.z + y.z * s.z) * k_scale,
+                                      (x.w * c.w + y.w * s.w) * k_scale);
+        *reinterpret_cast<float4*>(row + k_off + d) = lo;
+        *reinterpret_cast<float4*>(row + k_off + half + d) = hi;
+        *reinterpret_cast<float4*>(kd + d) = make_float4(lo.x * w, lo.y * w, lo.z * w, lo.w * w);
+        *reinterpret_cast<float4*>(kd + half + d) = make_float4(hi.x * w, hi.y * w, hi.z * w, hi.w * w);
+      } else {
+        const int d = 2 * half + 4 * (it - p4);
+        const float4 y = make_float4(ka[u].x * k_scale, ka[u].y * k_scale, ka[u].z * k_scale, ka[u].w * k_scale);
+        *reinterpret_cast<float4*>(row + k_off + d) = y;
+        *reinterpret_cast<float4*>(kd + d) = make_float4(y.x * w, y.y * w, y.z * w, y.w * w);
+      }
     }
   }
   ret_cp_wait<0>();
@@ -307,11 +346,13 @@ retention_chunk_state_kernel(float* proj, int ld, int q_off, int k_off, int v_of
     TileA A[MT];
 #pragma unroll
     for (int m = 0; m < MT; m++) A[m].set(v0[m0 + 16 * m], v0[m0 + 16 * m + 8], v4[m0 + 16 * m], v4[m0 + 16 * m + 8]);
+    constexpr int QS = NT % 2 == 0 ? 2 : 1;               // (column tiles at a time)
 #pragma unroll
-    for (int q = 0; q < NT; q++) {
-      const Split b0 = tf32_split(k0[n0 + 8 * q]), b1 = tf32_split(k4[n0 + 8 * q]);
+    for (int q = 0; q < NT; q += QS) {
+      Split b[QS][2];
 #pragma unroll
-      for (int m = 0; m < MT; m++) mma_split(acc[m][q], A[m], b0, b1);
+      for (int j = 0; j < QS; j++) { b[j][0] = tf32_split(k0[n0 + 8 * (q + j)]); b[j][1] = tf32_split(k4[n0 + 8 * (q + j)]); }
+      mma_split<MT, QS, NT>(acc, q, A, b);
     }
   }
   float* u = chunk_state + ((size_t)seg * H + h) * dv * dk;
@@ -328,34 +369,36 @@ retention_chunk_state_kernel(float* proj, int ld, int q_off, int k_off, int v_of
   if (tid == 0) chunk_decay[(size_t)seg * H + h] = pw[n];
 }
 
-// Kernel 3.  grid (chunks, H), 8 warps: warp (wr, wc) = (warp / 4, warp % 4) takes rows 32 wr .. + 31 and value columns
-// 8 NT wc ...  Shared memory: q, k and the state in rows of LDK, v in rows of LDV (4 above a multiple of 32: a fragment's
-// reads meet all banks); the scores take k's place.  The scores' fragments pair their columns 2 t and 2 t + 1 with the value
-// rows of the same numbers.
+// Kernel 3.  grid (chunks, H), 8 warps: warp (wr, wc) = (warp / 4, warp % 4) takes rows 32 wr .. + 31 and, of every 32 value
+// columns, the eight from 8 wc.  Shared memory, small enough for two blocks on an SM: q and k in rows of LDK (the scores take
+// k's place), and one more buffer that holds in turn up to 64 columns of the state in front of the chunk (rows of LDK), the
+// next 64, and the values (rows of LDV).  LDK and LDV are 4 above a multiple of 32: a fragment's reads meet all banks.  The
+// scores' fragments pair their columns 2 t and 2 t + 1 with the value rows of the same numbers.
 template <typename TO, int NT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 2)
 retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, int k_off, int v_off, int g_off,
                            const float* __restrict__ decay, float eps, const float* __restrict__ chunk_state,
                            const int* __restrict__ seg_start, const int* __restrict__ seg_seq, const int* __restrict__ seq_seg_start,
                            const int* __restrict__ start_pos, int H, int dk, int dv, int LDK, TO* __restrict__ out, int out_ld) {
   tlc_pdl(proj, chunk_state, out);
-  constexpr int DVP = 32 * NT, LDV = DVP + 4, LDP = RET_C + 4;
+  constexpr int DVP = 32 * NT, LDV = DVP + 4, LDP = RET_C + 4, PIECE = NT < 2 ? NT : 2;     // n-tiles of a piece of the state
   extern __shared__ __align__(16) float sh[];
   __shared__ float pw[RET_C + 1], red[RET_C][4];
-  float *qs = sh, *ks = qs + RET_C * LDK, *vs = ks + RET_C * max(LDK, LDP), *ss = vs + RET_C * LDV;
+  float *qs = sh, *ks = qs + RET_C * LDK, *buf = ks + RET_C * max(LDK, LDP);
   const int seg = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int t0 = seg_start[seg], n = min(seg_start[seg + 1] - t0, RET_C);
   const int b = seg_seq[seg];
   const bool empty = seg == seq_seg_start[b] && start_pos[b] == 0;         // nothing in front of the chunk
   const float a = decay[h];
-  const int dkp = (dk + 7) & ~7;
+  const int dkp = (dk + 7) & ~7, dk4 = dk >> 2, dv4 = dv >> 2;
+  const bool padded = n < RET_C || dk < dkp || dv < DVP;
   if (tid <= RET_C) pw[tid] = powf(a, (float)tid);
-  if (n < RET_C || dk < dkp || dv < DVP) {
-    const int total = RET_C * (LDK + max(LDK, LDP) + LDV) + DVP * LDK;
+  const int buf_floats = max(PIECE * 32 * LDK, RET_C * LDV);
+  if (padded) {                                           // rows and columns that no copy fills
+    const int total = RET_C * (LDK + max(LDK, LDP)) + buf_floats;
     for (int i = tid; i < total; i += 256) sh[i] = 0.f;
     __syncthreads();
   }
-  const int dk4 = dk >> 2, dv4 = dv >> 2;
   for (int i = tid; i < n * dk4; i += 256) {
     const int r = i / dk4, c = (i - r * dk4) << 2;
     const float* row = proj + (size_t)(t0 + r) * ld + (size_t)h * dk + c;
@@ -363,18 +406,25 @@ retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, in
     ret_cp16(ks + r * LDK + c, row + k_off);
   }
   ret_cp_commit();
-  if (!empty)
-    for (int i = tid; i < dv * dk4; i += 256) {
+  // value columns 32 p .. of the state (row v of it is a row of dk), PIECE * 32 of them; rows past dv stay as they are (they
+  // meet columns of the result that nobody stores)
+  auto load_state = [&](int p) {
+    const int first = 32 * p, rows = min(dv - first, 32 * PIECE);
+    for (int i = tid; i < rows * dk4; i += 256) {
       const int r = i / dk4, c = (i - r * dk4) << 2;
-      ret_cp16(ss + r * LDK + c, chunk_state + (((size_t)seg * H + h) * dv + r) * dk + c);
+      ret_cp16(buf + r * LDK + c, chunk_state + (((size_t)seg * H + h) * dv + first + r) * dk + c);
     }
-  ret_cp_commit();
-  for (int i = tid; i < n * dv4; i += 256) {
-    const int r = i / dv4, c = (i - r * dv4) << 2;
-    ret_cp16(vs + r * LDV + c, proj + (size_t)(t0 + r) * ld + v_off + (size_t)h * dv + c);
-  }
-  ret_cp_commit();
-  ret_cp_wait<2>();
+    ret_cp_commit();
+  };
+  auto load_values = [&]() {
+    for (int i = tid; i < n * dv4; i += 256) {
+      const int r = i / dv4, c = (i - r * dv4) << 2;
+      ret_cp16(buf + r * LDV + c, proj + (size_t)(t0 + r) * ld + v_off + (size_t)h * dv + c);
+    }
+    ret_cp_commit();
+  };
+  if (empty) load_values(); else load_state(0);
+  ret_cp_wait<1>();
   __syncthreads();
   const int g = lane >> 2, t = lane & 3, r0 = (warp >> 2) * 32, wc = warp & 3;
   // the scores of rows r0 .. + 31 and columns 16 wc .. + 15 (above the diagonal there is nothing)
@@ -385,8 +435,8 @@ retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, in
     for (int q = 0; q < 2; q++)
 #pragma unroll
       for (int e = 0; e < 4; e++) p[m][q][e] = 0.f;
-  const bool below = 16 * wc < r0 + 32;
-  if (below)
+  if (16 * wc < r0 + 32)
+#pragma unroll 2
     for (int d = 0; d < dkp; d += 8) {
       TileA A[2];
 #pragma unroll
@@ -394,13 +444,14 @@ retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, in
         const float* x = qs + (r0 + 16 * m + g) * LDK + d + t;
         A[m].set(x[0], x[8 * LDK], x[4], x[8 * LDK + 4]);
       }
+      Split kb[2][2];
 #pragma unroll
       for (int q = 0; q < 2; q++) {
         const float* y = ks + (16 * wc + 8 * q + g) * LDK + d + t;
-        const Split b0 = tf32_split(y[0]), b1 = tf32_split(y[4]);
-#pragma unroll
-        for (int m = 0; m < 2; m++) mma_split(p[m][q], A[m], b0, b1);
+        kb[q][0] = tf32_split(y[0]);
+        kb[q][1] = tf32_split(y[4]);
       }
+      mma_split<2, 2, 2>(p, 0, A, kb);
     }
   __syncthreads();                                        // k has been read
   float* ps = ks;
@@ -409,12 +460,10 @@ retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, in
 #pragma unroll
     for (int q = 0; q < 2; q++)
 #pragma unroll
-      for (int e = 0; e < 4; e++) {
-        const int i = r0 + 16 * m + g + (e >> 1) * 8, j = 16 * wc + 8 * q + 2 * t + (e & 1);
-        ps[i * LDP + j] = j <= i ? p[m][q][e] * pw[i - j] : 0.f;
+      for (int e = 0; e < 4; e += 2) {
+        const int i = r0 + 16 * m + g + (e >> 1) * 8, j = 16 * wc + 8 * q + 2 * t;
+        *reinterpret_cast<float2*>(ps + i * LDP + j) = make_float2(j <= i ? p[m][q][e] * pw[i - j] : 0.f, j + 1 <= i ? p[m][q][e + 1] * pw[i - j - 1] : 0.f);
       }
-  ret_cp_wait<1>();
-  __syncthreads();                                        // the scores and the state are there
   float acc[2][NT][4];
 #pragma unroll
   for (int m = 0; m < 2; m++)
@@ -422,21 +471,37 @@ retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, in
     for (int q = 0; q < NT; q++)
 #pragma unroll
       for (int e = 0; e < 4; e++) acc[m][q][e] = 0.f;
-  const int c0 = wc * 8 * NT;
   if (!empty) {
-    for (int d = 0; d < dkp; d += 8) {
-      TileA A[2];
 #pragma unroll
-      for (int m = 0; m < 2; m++) {
-        const float* x = qs + (r0 + 16 * m + g) * LDK + d + t;
-        A[m].set(x[0], x[8 * LDK], x[4], x[8 * LDK + 4]);
+    for (int q0 = 0; q0 < NT; q0 += PIECE) {
+      ret_cp_wait<0>();
+      __syncthreads();                                    // this piece of the state has landed
+#pragma unroll 2
+      for (int d = 0; d < dkp; d += 8) {
+        TileA A[2];
+#pragma unroll
+        for (int m = 0; m < 2; m++) {
+          const float* x = qs + (r0 + 16 * m + g) * LDK + d + t;
+          A[m].set(x[0], x[8 * LDK], x[4], x[8 * LDK + 4]);
+        }
+        Split sb[PIECE][2];
+#pragma unroll
+        for (int q = 0; q < PIECE; q++) {
+          const float* y = buf + (32 * q + 8 * wc + g) * LDK + d + t;
+          sb[q][0] = tf32_split(y[0]);
+          sb[q][1] = tf32_split(y[4]);
+        }
+        mma_split<2, PIECE, NT>(acc, q0, A, sb);
       }
-#pragma unroll
-      for (int q = 0; q < NT; q++) {
-        const float* y = ss + (c0 + 8 * q + g) * LDK + d + t;
-        const Split b0 = tf32_split(y[0]), b1 = tf32_split(y[4]);
-#pragma unroll
-        for (int m = 0; m < 2; m++) mma_split(acc[m][q], A[m], b0, b1);
+      __syncthreads();                                    // the buffer has been read
+      if (q0 + PIECE < NT) {
+        load_state(q0 + PIECE);
+      } else {
+        if (padded) {
+          for (int i = tid; i < buf_floats; i += 256) buf[i] = 0.f;
+          __syncthreads();
+        }
+        load_values();
       }
     }
 #pragma unroll
@@ -450,7 +515,7 @@ retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, in
     }
   }
   ret_cp_wait<0>();
-  __syncthreads();
+  __syncthreads();                                        // the values and every warp's scores are there
   const int last = min(r0 + 32, (n + 7) & ~7);            // later columns meet no row of this warp
   for (int j = 0; j < last; j += 8) {
     TileA A[2];
@@ -460,13 +525,14 @@ retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, in
       const float2 y = *reinterpret_cast<const float2*>(ps + (r0 + 16 * m + g + 8) * LDP + j + 2 * t);
       A[m].set(x.x, y.x, x.y, y.y);
     }
+    Split vb[NT][2];
 #pragma unroll
     for (int q = 0; q < NT; q++) {
-      const float* y = vs + (j + 2 * t) * LDV + c0 + 8 * q + g;
-      const Split b0 = tf32_split(y[0]), b1 = tf32_split(y[LDV]);
-#pragma unroll
-      for (int m = 0; m < 2; m++) mma_split(acc[m][q], A[m], b0, b1);
+      const float* y = buf + (j + 2 * t) * LDV + 32 * q + 8 * wc + g;
+      vb[q][0] = tf32_split(y[0]);
+      vb[q][1] = tf32_split(y[LDV]);
     }
+    mma_split<2, NT, NT>(acc, 0, A, vb);
   }
   // the head's norm over all value columns (four warps share a row), then the gate
 #pragma unroll
@@ -474,6 +540,7 @@ retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, in
     float s0 = 0.f, s1 = 0.f;
 #pragma unroll
     for (int q = 0; q < NT; q++) {
+      if (32 * q + 8 * wc + 2 * t >= dv) continue;        // (what stands in columns past the head's is of no account)
       s0 += acc[m][q][0] * acc[m][q][0] + acc[m][q][1] * acc[m][q][1];
       s1 += acc[m][q][2] * acc[m][q][2] + acc[m][q][3] * acc[m][q][3];
     }
@@ -482,6 +549,7 @@ retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, in
     if (t == 0) { red[r0 + 16 * m + g][wc] = s0; red[r0 + 16 * m + g + 8][wc] = s1; }
   }
   __syncthreads();
+  const bool pairs = out_ld % 2 == 0 && (uintptr_t)out % 4 == 0;
 #pragma unroll
   for (int m = 0; m < 2; m++)
 #pragma unroll
@@ -493,11 +561,16 @@ retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, in
       TO* o = out + (size_t)(t0 + r) * out_ld + (size_t)h * dv;
 #pragma unroll
       for (int q = 0; q < NT; q++) {
-        const int v = c0 + 8 * q + 2 * t;
+        const int v = 32 * q + 8 * wc + 2 * t;
         if (v < dv) {                                     // (dv is a multiple of 4)
           const float2 z = *reinterpret_cast<const float2*>(gate + v);
-          o[v] = from_f32<TO>(acc[m][q][2 * e] * inv * silu_of<sizeof(TO) == 2>(z.x));
-          o[v + 1] = from_f32<TO>(acc[m][q][2 * e + 1] * inv * silu_of<sizeof(TO) == 2>(z.y));
+          const float y0 = acc[m][q][2 * e] * inv * silu_of<sizeof(TO) == 2>(z.x), y1 = acc[m][q][2 * e + 1] * inv * silu_of<sizeof(TO) == 2>(z.y);
+          if (sizeof(TO) == 2 && pairs) {
+            *reinterpret_cast<__nv_bfloat162*>(o + v) = __floats2bfloat162_rn(y0, y1);
+          } else {
+            o[v] = from_f32<TO>(y0);
+            o[v + 1] = from_f32<TO>(y1);
+          }
         }
       }
     }
@@ -506,7 +579,8 @@ retention_chunk_out_kernel(const float* __restrict__ proj, int ld, int q_off, in
 static int ret_ldk(int dk) { return (dk + 31) / 32 * 32 + 4; }
 static size_t ret_out_smem(int dk, int dvp) {
   const int ldk = ret_ldk(dk);
-  return (size_t)(RET_C * (ldk + (ldk > RET_C + 4 ? ldk : RET_C + 4) + dvp + 4) + dvp * ldk) * sizeof(float);
+  const int piece = (dvp < 64 ? dvp : 64) * ldk, values = RET_C * (dvp + 4);
+  return (size_t)(RET_C * (ldk + (ldk > RET_C + 4 ? ldk : RET_C + 4)) + (piece > values ? piece : values)) * sizeof(float);
 }
 static size_t ret_state_smem(int dk, int dv, int rope_dim) {
   return (size_t)RET_C * ((dk + 31) / 32 * 32 + 8 + (dv + 31) / 32 * 32 + 8 + rope_dim) * sizeof(float);

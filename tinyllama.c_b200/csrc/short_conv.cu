@@ -154,7 +154,18 @@ rmsnorm_conv_rows_kernel(const float* __restrict__ x, const float* __restrict__ 
     float ss = 0.f;
     if (t >= 0 && t < n_rows) {
       const float* xr = x + (size_t)t * D;
-      for (int d = lane * V; d < D; d += 32 * V) {
+      constexpr int U = 8;                              // (loads issued together)
+      int d = lane * V;
+      for (; d + (U - 1) * 32 * V < D; d += U * 32 * V) {
+        Vec<V> v[U];
+#pragma unroll
+        for (int u = 0; u < U; u++) v[u] = Vec<V>::ld(xr + d + u * 32 * V);
+#pragma unroll
+        for (int u = 0; u < U; u++)
+#pragma unroll
+          for (int e = 0; e < V; e++) ss = fmaf(v[u].v[e], v[u].v[e], ss);
+      }
+      for (; d < D; d += 32 * V) {
         const Vec<V> v = Vec<V>::ld(xr + d);
 #pragma unroll
         for (int e = 0; e < V; e++) ss = fmaf(v.v[e], v.v[e], ss);
@@ -166,8 +177,10 @@ rmsnorm_conv_rows_kernel(const float* __restrict__ x, const float* __restrict__ 
   __syncthreads();
   for (int d = threadIdx.x * V; d < D; d += 256 * V) {
     const Vec<V> gv = Vec<V>::ld(g + d);
-    auto normed = [&](int t, float inv) {
-      Vec<V> v = Vec<V>::ld(x + (size_t)t * D + d);
+    Vec<V> rows[CONV_R];                                // (loads issued together)
+#pragma unroll
+    for (int r = 0; r < CONV_R; r++) rows[r] = t0 + r < n_rows ? Vec<V>::ld(x + (size_t)(t0 + r) * D + d) : vzero<V>();
+    auto scaled = [&](Vec<V> v, float inv) {
 #pragma unroll
       for (int e = 0; e < V; e++) v.v[e] = v.v[e] * inv * gv.v[e];
       return v;
@@ -181,7 +194,7 @@ rmsnorm_conv_rows_kernel(const float* __restrict__ x, const float* __restrict__ 
     for (int j = 0; j < Window<KT, V>::N; j++) {
       if (j < K - 1) {
         const int back = K - 1 - j, i = s.i[0] - back;
-        if (i >= 0) win.win[j] = normed(t0 - back, s_inv[j]);
+        if (i >= 0) win.win[j] = scaled(Vec<V>::ld(x + (size_t)(t0 - back) * D + d), s_inv[j]);
         else if (s.has[0]) win.win[j] = Vec<V>::ld(state + ((size_t)s.slot[0] * (K - 1) + (K - 1 + i)) * D + d);
       }
     }
@@ -193,7 +206,7 @@ rmsnorm_conv_rows_kernel(const float* __restrict__ x, const float* __restrict__ 
         if (s.has[r]) win.load(state + (size_t)s.slot[r] * (K - 1) * D + d, D, K);
         else win.clear();
       }
-      const Vec<V> cur = normed(t, s_inv[K - 1 + r]);
+      const Vec<V> cur = scaled(rows[r], s_inv[K - 1 + r]);
       conv_step<KT, V>(win, taps, cur, w + d, D, K, cur).st(out + (size_t)t * D + d);
       if (write_state && s.last[r]) win.store(state + (size_t)s.slot[r] * (K - 1) * D + d, D, K);
     }
