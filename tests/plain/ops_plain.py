@@ -58,15 +58,18 @@ def _gate_up(gate_up, interleaved):
     return r[:, :, 0, :].reshape(-1, F), r[:, :, 1, :].reshape(-1, F)
 
 
-def linear_swiglu(a, w, out, colscale=None, colbias=None, act="silu"):
+def linear_swiglu(a, w, out, colscale=None, colbias=None, act="silu", limit=0.0, alpha=1.0):
     gu = torch.empty((a.shape[0], w.shape[0]), dtype=torch.float64)
     linear(a, w, gu, colscale, colbias)
-    glu(gu, out, act, interleaved=True)
+    glu(gu, out, act, interleaved=True, limit=limit, alpha=alpha)
 
 
-def glu(gate_up, out, act="silu", interleaved=False):
+def glu(gate_up, out, act="silu", interleaved=False, limit=0.0, alpha=1.0):
     g, u = _gate_up(gate_up, interleaved)
-    if act == "gelu_tanh":
+    if act == "swish_clamped":
+        g, u = torch.clamp(g, max=limit), torch.clamp(u, -limit, limit)
+        a, u = g / (1.0 + torch.exp(-alpha * g)), u + 1.0
+    elif act == "gelu_tanh":
         a = 0.5 * g * (1.0 + torch.tanh(0.7978845608028654 * (g + 0.044715 * g ** 3)))
     else:
         a = g / (1.0 + torch.exp(-g))
@@ -120,7 +123,7 @@ def rope_kv_store(qkv, q_off, k_off, v_off, q_out, k_pages, v_pages, inv_freq, p
 
 def attention(q, k_pages, v_pages, block_table, positions, row_seq, slots, out, H, KV, hd, scale, window=0,
               decode_max_keys=0, cu_seqlens=None, start_pos=None, max_keys=0, max_blocks=0, key_ranges=0, softcap=0.0, sink=False,
-              keep_first=0, sink_values=None):
+              keep_first=0, sink_values=None, chunk=0, head_gate=None):
     T = q.shape[0]
     res = torch.zeros((T, H, hd), dtype=torch.float64)
     qf = _f(q).reshape(T, H, hd)
@@ -129,6 +132,8 @@ def attention(q, k_pages, v_pages, block_table, positions, row_seq, slots, out, 
         table = block_table[int(slots[int(row_seq[t])])]
         n_keys = p + 1
         start = n_keys - window if (window and n_keys > window) else 0
+        if chunk:                                                   # only keys of the row's own chunk
+            start = max(start, p // chunk * chunk)
         idx = torch.arange(start, n_keys)
         if window and keep_first and start > 0:                     # the sequence's first keys stay visible
             idx = torch.cat([torch.arange(0, min(keep_first, start)), idx])
@@ -146,6 +151,8 @@ def attention(q, k_pages, v_pages, block_table, positions, row_seq, slots, out, 
             else:
                 pr = torch.softmax(sc, dim=0)
             res[t, h] = pr @ V[:, g]
+            if head_gate is not None:
+                res[t, h] *= 1.0 / (1.0 + torch.exp(-_f(head_gate[t, h])))
     out.copy_(res.reshape(T, H * hd).to(out.dtype))
 
 

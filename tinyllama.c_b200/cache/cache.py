@@ -8,10 +8,10 @@ one by one (graph.c:343-357; falcon_h1.c:136-147) and serves one sequence per se
 
 * a *slot* belongs to one live sequence and records its length; slots are handed back
   when the sequence ends and reused by later ones;
-* layers whose mixers ask for keys/values with the same (kv heads, head size, window) form
+* layers whose mixers ask for keys/values with the same (kv heads, head size, window, chunk) form
   a *group* with one page pool [layers, pages, kv heads, 64, head size] and one block
-  table [slots, pages per slot]; a windowed group gives back pages that fell out of every
-  future query's window (except those that hold the first positions a request says stay visible);
+  table [slots, pages per slot]; a windowed (or chunked) group gives back pages that fell out of every
+  future query's window (or belong to chunks that are over; except those that hold the first positions a request says stay visible);
 * every fixed-size state request (same key and shape) forms a group [layers, slots, *shape];
   a sequence at position 0 is treated as all-zero by the kernels, so nothing is cleared
   on reuse.
@@ -33,6 +33,11 @@ PAGE = 64
 
 def pages_for(n_tokens: int) -> int:
     return (int(n_tokens) + PAGE - 1) // PAGE
+
+
+def _pages_signature(r: KVRequest) -> tuple:
+    """Requests that agree in this share a group: the same pages are held and given back at the same time."""
+    return (r.kv_heads, r.head_dim, r.window, r.values, r.keep_first if r.window else 0, int(r.chunk or 0))
 
 
 @dataclass
@@ -77,10 +82,8 @@ class Cache:
         for cid in sorted(requests):
             for req in requests[cid]:
                 if isinstance(req, KVRequest):
-                    sig = (req.kv_heads, req.head_dim, req.window, req.values, req.keep_first if req.window else 0)
-                    gi = next((i for i, g in enumerate(self.kv_groups)
-                               if (g.request.kv_heads, g.request.head_dim, g.request.window, g.request.values,
-                                   g.request.keep_first if g.request.window else 0) == sig), None)
+                    sig = _pages_signature(req)
+                    gi = next((i for i, g in enumerate(self.kv_groups) if _pages_signature(g.request) == sig), None)
                     if gi is None:
                         self.kv_groups.append(_KVGroup(req, [], None, None, None, None,
                                                        IndexPool(self.n_pages, "cache page"),
@@ -169,13 +172,14 @@ class Cache:
         return start
 
     def commit(self, slot: int, n_new: int) -> None:
-        """The step stored n_new positions; windowed groups give back pages no later query can see."""
+        """The step stored n_new positions; windowed and chunked groups give back pages no later query can see."""
         self.seq_len[slot] += n_new
         L = self.seq_len[slot]
         for g in self.kv_groups:
-            w = g.request.window
-            if w:
-                first_needed = max(0, L + 1 - w) // PAGE       # the next query at position L sees keys >= L+1-w
+            w, c = g.request.window, g.request.chunk
+            if w or c:
+                # the next query at position L sees keys >= L+1-w, or the keys of its own chunk
+                first_needed = max(L + 1 - w if w else 0, L - L % c if c else 0, 0) // PAGE
                 have = g.pages_of[slot]
                 kept = pages_for(max(0, g.request.keep_first))  # pages with positions that every later query still sees
                 for i in range(kept, min(first_needed, len(have))):

@@ -6,3 +6,4 @@ from .porarax import PoraraxConfig  # noqa: F401
 from .sogazen import SogazenConfig  # noqa: F401
 from .kimutar import KimutarConfig  # noqa: F401
 from .kefetar import KefetarConfig  # noqa: F401
+from .fobatar import FobatarConfig  # noqa: F401

@@ -173,8 +173,8 @@ attention_warp_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, co
                       const int* __restrict__ block_table, int max_pages, const int* __restrict__ positions,
                       const int* __restrict__ row_seq, const int* __restrict__ slots, T* __restrict__ out, int H, int KV,
                       int hd, float scale, int window, int out_ld, float softcap, int sink, int keep_first,
-                      const float* __restrict__ sink_values) {
-  tlc_pdl(q, k_pages, v_pages, out);
+                      const float* __restrict__ sink_values, int chunk, const float* __restrict__ head_gate, int gate_ld) {
+  tlc_pdl(q, k_pages, v_pages, out, head_gate);
   extern __shared__ float qs_all[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
@@ -188,7 +188,7 @@ attention_warp_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, co
   for (int d = lane; d < hd; d += 32) qs[d] = to_f32(qr[d]) * scale;
   __syncwarp();
   const int n_keys = pos + 1;
-  const int start = (window > 0 && n_keys > window) ? n_keys - window : 0;
+  const int start = tlc_first_key(pos, window, chunk);
   float m = -INFINITY, l = 0.f;
   float acc[ATT_MAXD];
 #pragma unroll
@@ -236,7 +236,7 @@ attention_warp_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, co
 #pragma unroll
     for (int i = 0; i < ATT_MAXD; i++) acc[i] *= corr;
   }
-  const float inv = 1.0f / l;
+  const float inv = tlc_head_gate(head_gate, gate_ld, t, h) / l;
   T* o = out + (size_t)t * out_ld + (size_t)h * hd;
 #pragma unroll
   for (int i = 0; i < ATT_MAXD; i++) {
@@ -248,8 +248,8 @@ attention_warp_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, co
 extern "C" int tlc_attention(const void* q, int dtype, const void* k_pages, const void* v_pages,
                              const int* block_table, int max_pages, const int* positions, const int* row_seq,
                              const int* slots, void* out, int T, int H, int KV, int hd, float scale, int window,
-                             int out_ld, float softcap, int sink, int keep_first, const float* sink_values,
-                             cudaStream_t stream) {
+                             int out_ld, float softcap, int sink, int keep_first, const float* sink_values, int chunk,
+                             const float* head_gate, int gate_ld, cudaStream_t stream) {
   if (T == 0) return 0;
   if (out_ld <= 0) out_ld = H * hd;                      // elements between rows of out (0: dense)
   TLC_REQUIRE(KV > 0 && H % KV == 0, "attention: %d heads are not a multiple of %d key/value heads", H, KV);
@@ -258,7 +258,7 @@ extern "C" int tlc_attention(const void* q, int dtype, const void* k_pages, cons
   const size_t smem = (size_t)4 * hd * sizeof(float);
   TLC_DISPATCH_DTYPE(dtype, TT, tlc_launch(attention_warp_kernel<TT>, dim3(grid), dim3(128), smem, stream, 
       (const TT*)q, (const TT*)k_pages, (const TT*)v_pages, block_table, max_pages, positions, row_seq, slots, (TT*)out,
-      H, KV, hd, scale, window, out_ld, softcap, sink, keep_first, sink_values));
+      H, KV, hd, scale, window, out_ld, softcap, sink, keep_first, sink_values, chunk, head_gate, gate_ld));
   TLC_CHECK_LAUNCH("attention");
   return 0;
 }
@@ -270,6 +270,8 @@ extern "C" int tlc_attention(const void* q, int dtype, const void* k_pages, cons
 // output with its running maximum and sum; a second kernel merges the splits.  The split count
 // of the grid is an upper bound from the host; a block whose keys lie past the row's length or
 // before its window exits at once, so the same launch serves any lengths (and a captured graph).
+// With a window or chunks the splits are counted from the page of the first visible key (unless the
+// sequence's first keys stay visible), so that the bound is what a row sees, not what it has.
 #define DEC_KEYS 128
 #define DEC_MAXG 8
 template <typename T>
@@ -278,16 +280,16 @@ attention_decode_partial_kernel(const T* __restrict__ q, const T* __restrict__ k
                                 const int* __restrict__ block_table, int max_pages, const int* __restrict__ positions,
                                 const int* __restrict__ row_seq, const int* __restrict__ slots, float* __restrict__ part_o,
                                 float* __restrict__ part_ml, int H, int KV, int hd, float scale, int window, int n_splits,
-                                float softcap, int keep_first) {
+                                float softcap, int keep_first, int chunk) {
   tlc_pdl(q, k_pages, v_pages, part_o, part_ml);
   extern __shared__ float sh[];
   const int t = blockIdx.x, g = blockIdx.y, split = blockIdx.z;
   const int G = H / KV;
   const int pos = positions[t];
   const int n_keys = pos + 1;
-  const int start = (window > 0 && n_keys > window) ? n_keys - window : 0;
-  const int k0 = split * DEC_KEYS;
+  const int start = tlc_first_key(pos, window, chunk);
   const int kept = min(max(keep_first, 0), start);      // with a window, the sequence's first keys stay visible
+  const int k0 = (kept > 0 ? 0 : start / TLC_PAGE * TLC_PAGE) + split * DEC_KEYS;
   float* ml = part_ml + (((size_t)t * H + (size_t)g * G) * n_splits + split) * 2;   // + hg * n_splits * 2
   if (k0 >= n_keys || (k0 + DEC_KEYS <= start && k0 >= kept)) {
     if (threadIdx.x < G) { ml[(size_t)threadIdx.x * n_splits * 2] = -INFINITY; ml[(size_t)threadIdx.x * n_splits * 2 + 1] = 0.f; }
@@ -357,7 +359,7 @@ attention_decode_partial_vec_kernel(const __nv_bfloat16* __restrict__ q, const _
                                     int max_pages, const int* __restrict__ positions, const int* __restrict__ row_seq,
                                     const int* __restrict__ slots, float* __restrict__ part_o,
                                     float* __restrict__ part_ml, int H, int KV, float scale, int window, int n_splits,
-                                    float softcap, int keep_first) {
+                                    float softcap, int keep_first, int chunk) {
   // Keys of earlier positions were stored by earlier steps; only the row at the query's own
   // position is written by the kernel before this one.  Everything else is fetched before the
   // wait on that kernel (see tlc_pdl).
@@ -369,9 +371,9 @@ attention_decode_partial_vec_kernel(const __nv_bfloat16* __restrict__ q, const _
   const int G = H / KV;
   const int pos = positions[t];
   const int n_keys = pos + 1;
-  const int start = (window > 0 && n_keys > window) ? n_keys - window : 0;
-  const int k0 = split * DEC_KEYS;
+  const int start = tlc_first_key(pos, window, chunk);
   const int kept = min(max(keep_first, 0), start);      // with a window, the sequence's first keys stay visible
+  const int k0 = (kept > 0 ? 0 : start / TLC_PAGE * TLC_PAGE) + split * DEC_KEYS;
   float* ml = part_ml + (((size_t)t * H + (size_t)g * G) * n_splits + split) * 2;
   if (k0 >= n_keys || (k0 + DEC_KEYS <= start && k0 >= kept)) {
     tlc_wait(ml);
@@ -529,8 +531,9 @@ attention_decode_partial_vec_kernel(const __nv_bfloat16* __restrict__ q, const _
 template <typename T>
 __global__ void attention_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                               T* __restrict__ out, int hd, int n_splits, int H, int out_ld, int sink,
-                                              const float* __restrict__ sink_values) {
-  tlc_pdl(part_o, part_ml, out);
+                                              const float* __restrict__ sink_values, const float* __restrict__ head_gate,
+                                              int gate_ld) {
+  tlc_pdl(part_o, part_ml, out, head_gate);
   const size_t th = blockIdx.x;                       // row * H + head
   T* orow = out + (th / H) * (size_t)out_ld + (th % H) * (size_t)hd;
   const float* ml = part_ml + th * n_splits * 2;
@@ -539,7 +542,7 @@ __global__ void attention_decode_merge_kernel(const float* __restrict__ part_o, 
   for (int s = 0; s < n_splits; s++) m = fmaxf(m, ml[2 * s]);
   float l = sink ? expf(sv - m) : 0.f;
   for (int s = 0; s < n_splits; s++) if (ml[2 * s + 1] > 0.f) l += ml[2 * s + 1] * expf(ml[2 * s] - m);
-  const float inv = 1.0f / l;
+  const float inv = tlc_head_gate(head_gate, gate_ld, (int)(th / H), (int)(th % H)) / l;
   for (int d = threadIdx.x; d < hd; d += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < n_splits; s++)
@@ -548,12 +551,14 @@ __global__ void attention_decode_merge_kernel(const float* __restrict__ part_o, 
   }
 }
 
-// scratch: part_o [T, H, n_splits, hd] and part_ml [T, H, n_splits, 2] floats, n_splits = ceil(max_keys / 128)
+// scratch: part_o [T, H, n_splits, hd] and part_ml [T, H, n_splits, 2] floats, n_splits = ceil(max_keys / 128);
+// max_keys: the longest sequence, or with a window or chunks (and keep_first 0) their size + 63 where that is less
 extern "C" int tlc_attention_decode(const void* q, int dtype, const void* k_pages, const void* v_pages,
                                     const int* block_table, int max_pages, const int* positions, const int* row_seq,
                                     const int* slots, void* out, float* part_o, float* part_ml, int T, int H, int KV,
                                     int hd, float scale, int window, int max_keys, int out_ld, float softcap, int sink,
-                                    int keep_first, const float* sink_values, cudaStream_t stream) {
+                                    int keep_first, const float* sink_values, int chunk, const float* head_gate, int gate_ld,
+                                    cudaStream_t stream) {
   if (T == 0) return 0;
   if (out_ld <= 0) out_ld = H * hd;                      // elements between rows of out (0: dense)
   TLC_REQUIRE(KV > 0 && H % KV == 0, "attention: %d heads are not a multiple of %d key/value heads", H, KV);
@@ -570,12 +575,12 @@ extern "C" int tlc_attention_decode(const void* q, int dtype, const void* k_page
     if (vsmem <= 48 * 1024) {
       const __nv_bfloat16 *qp = (const __nv_bfloat16*)q, *kp = (const __nv_bfloat16*)k_pages, *vp = (const __nv_bfloat16*)v_pages;
       if (hd == 64)
-        tlc_launch(attention_decode_partial_vec_kernel<64>, dim3(grid), dim3(DEC_KEYS), vsmem, stream, qp, kp, vp, block_table, max_pages, positions, row_seq, slots, part_o, part_ml, H, KV, scale, window, n_splits, softcap, keep_first);
+        tlc_launch(attention_decode_partial_vec_kernel<64>, dim3(grid), dim3(DEC_KEYS), vsmem, stream, qp, kp, vp, block_table, max_pages, positions, row_seq, slots, part_o, part_ml, H, KV, scale, window, n_splits, softcap, keep_first, chunk);
       else if (hd == 128)
-        tlc_launch(attention_decode_partial_vec_kernel<128>, dim3(grid), dim3(DEC_KEYS), vsmem, stream, qp, kp, vp, block_table, max_pages, positions, row_seq, slots, part_o, part_ml, H, KV, scale, window, n_splits, softcap, keep_first);
+        tlc_launch(attention_decode_partial_vec_kernel<128>, dim3(grid), dim3(DEC_KEYS), vsmem, stream, qp, kp, vp, block_table, max_pages, positions, row_seq, slots, part_o, part_ml, H, KV, scale, window, n_splits, softcap, keep_first, chunk);
       else
-        tlc_launch(attention_decode_partial_vec_kernel<256>, dim3(grid), dim3(DEC_KEYS), vsmem, stream, qp, kp, vp, block_table, max_pages, positions, row_seq, slots, part_o, part_ml, H, KV, scale, window, n_splits, softcap, keep_first);
-      tlc_launch(attention_decode_merge_kernel<__nv_bfloat16>, dim3(T * H), dim3(128), 0, stream, part_o, part_ml, (__nv_bfloat16*)out, hd, n_splits, H, out_ld, sink, sink_values);
+        tlc_launch(attention_decode_partial_vec_kernel<256>, dim3(grid), dim3(DEC_KEYS), vsmem, stream, qp, kp, vp, block_table, max_pages, positions, row_seq, slots, part_o, part_ml, H, KV, scale, window, n_splits, softcap, keep_first, chunk);
+      tlc_launch(attention_decode_merge_kernel<__nv_bfloat16>, dim3(T * H), dim3(128), 0, stream, part_o, part_ml, (__nv_bfloat16*)out, hd, n_splits, H, out_ld, sink, sink_values, head_gate, gate_ld);
       TLC_CHECK_LAUNCH("attention(decode)");
       return 0;
     }
@@ -583,8 +588,8 @@ extern "C" int tlc_attention_decode(const void* q, int dtype, const void* k_page
   TLC_DISPATCH_DTYPE(dtype, TT, {
     tlc_launch(attention_decode_partial_kernel<TT>, dim3(grid), dim3(DEC_KEYS), smem, stream, 
         (const TT*)q, (const TT*)k_pages, (const TT*)v_pages, block_table, max_pages, positions, row_seq, slots, part_o,
-        part_ml, H, KV, hd, scale, window, n_splits, softcap, keep_first);
-    tlc_launch(attention_decode_merge_kernel<TT>, dim3(T * H), dim3(128), 0, stream, part_o, part_ml, (TT*)out, hd, n_splits, H, out_ld, sink, sink_values);
+        part_ml, H, KV, hd, scale, window, n_splits, softcap, keep_first, chunk);
+    tlc_launch(attention_decode_merge_kernel<TT>, dim3(T * H), dim3(128), 0, stream, part_o, part_ml, (TT*)out, hd, n_splits, H, out_ld, sink, sink_values, head_gate, gate_ld);
   });
   TLC_CHECK_LAUNCH("attention(decode)");
   return 0;
@@ -628,5 +633,5 @@ extern "C" int tlc_attention_decode_no_alloc(const void* q, int dtype, const voi
   float* part_o = g_decode_scratch_addr[dev];
   float* part_ml = part_o + (size_t)T * H * n_splits * hd;
   return tlc_attention_decode(q, dtype, k_pages, v_pages, block_table, max_pages, positions, row_seq, slots, out, part_o,
-                              part_ml, T, H, KV, hd, scale, window, max_keys, 0, 0.f, 0, 0, nullptr, stream);
+                              part_ml, T, H, KV, hd, scale, window, max_keys, 0, 0.f, 0, 0, nullptr, 0, nullptr, 0, stream);
 }

@@ -86,7 +86,8 @@ attention_decode_fused_kernel(const float* __restrict__ qkv, int ld, int q_off, 
                             float* __restrict__ part_ml, unsigned* __restrict__ arrivals,
                             __nv_bfloat16* __restrict__ out, int H, int KV, float scale, int window, int n_splits,
                             int passes, int out_ld, float softcap, int sink, int keep_first,
-                            const float* __restrict__ sink_values) {
+                            const float* __restrict__ sink_values, int chunk, const float* __restrict__ head_gate,
+                            int gate_ld) {
   // Keys and values of earlier positions were stored by earlier steps and are fetched before the
   // wait on the previous kernel; the row's own projection is read after it.
   asm volatile("griddepcontrol.launch_dependents;");
@@ -99,11 +100,12 @@ attention_decode_fused_kernel(const float* __restrict__ qkv, int ld, int q_off, 
   const int G = H / KV;
   const int pos = positions[t];
   const int n_keys = pos + 1;
-  const int start = (window > 0 && n_keys > window) ? n_keys - window : 0;
+  const int start = tlc_first_key(pos, window, chunk);
   const int kept = min(max(keep_first, 0), start);    // with a window, the sequence's first keys stay visible
   const int round = FM_NW * CK;              // keys of one round of the block's warps
   const int span = round * passes;           // keys of this block
-  const int kbase = split * span;
+  // with a window or chunks the splits are counted from the page of the first visible key: the grid is for what a row sees
+  const int kbase = (kept > 0 ? 0 : start / TLC_PAGE * TLC_PAGE) + split * span;
   const int n_pg = (span + TLC_PAGE - 1) / TLC_PAGE;
   const int smem_floats = L::FIXED / 4;
   float* ml = part_ml + (((size_t)t * H + (size_t)g * G) * n_splits + split) * 2;
@@ -162,7 +164,7 @@ attention_decode_fused_kernel(const float* __restrict__ qkv, int ld, int q_off, 
     };
 #pragma unroll
     for (int s = 0; s < STAGES; s++) issue(j_first + s);
-    tlc_wait(qkv, k_pages, v_pages, part_o, ml, out);
+    tlc_wait(qkv, k_pages, v_pages, part_o, ml, out, head_gate);
     // rotation: the thread of dim d turns that dim of every query head of the group and of the key;
     // all of its loads are issued before the first use
     for (int d = tid; d < HD; d += FM_NT) {
@@ -336,7 +338,8 @@ attention_decode_fused_kernel(const float* __restrict__ qkv, int ld, int q_off, 
       }
       const size_t th = (size_t)t * H + (size_t)g * G + hg;
       if (n_splits == 1) {
-        out[(size_t)t * out_ld + ((size_t)g * G + hg) * HD + d] = __float2bfloat16_rn(o * (1.0f / l));
+        out[(size_t)t * out_ld + ((size_t)g * G + hg) * HD + d] =
+            __float2bfloat16_rn(o * (tlc_head_gate(head_gate, gate_ld, t, g * G + hg) / l));
       } else {
         part_o[(th * n_splits + split) * HD + d] = o;
         if (d == 0) { ml[(size_t)hg * n_splits * 2] = M; ml[(size_t)hg * n_splits * 2 + 1] = l; }
@@ -354,7 +357,7 @@ attention_decode_fused_kernel(const float* __restrict__ qkv, int ld, int q_off, 
   __syncthreads();
   if (!s_last) return;
   __threadfence();
-  attention_merge_splits<HD, FM_NT>(part_o, part_ml, out, reinterpret_cast<float*>(smraw), smem_floats, t, g, G, H, n_splits, out_ld, sink, sink_values);
+  attention_merge_splits<HD, FM_NT>(part_o, part_ml, out, reinterpret_cast<float*>(smraw), smem_floats, t, g, G, H, n_splits, out_ld, sink, sink_values, head_gate, gate_ld);
 }
 
 int g_fused_passes = 0;       // > 0: rounds a block takes, for tests (0: chosen from the grid)
@@ -386,13 +389,17 @@ extern "C" int tlc_attention_decode_fused_ok(int H, int KV, int hd) {
 // v_off.  scratch: part_o [T, H, n_splits, hd], part_ml [T, H, n_splits, 2] floats with
 // n_splits <= ceil(max_keys / 128); arrivals: T * KV counters, zero before the first call.  softcap > 0: score <-
 // softcap * tanh(score / softcap) after the scale; sink: one more term of score 0 in the softmax's denominator.
+// max_keys: the longest sequence after the step, or with a window or chunks (and keep_first 0) their size + 63 where
+// that is less.  chunk > 0: a row sees the keys of its own chunk of that many positions.  head_gate [T, H] float (rows of
+// gate_ld values, NULL: none): a head's result is multiplied by the sigmoid of its number.
 extern "C" int tlc_attention_decode_fused(const float* qkv, int ld, int q_off, int k_off, int v_off, void* k_pages,
                                         void* v_pages, const float* inv_freq, int rope_dim, int write_kv,
                                         const int* block_table, int max_pages, const int* positions,
                                         const int* row_seq, const int* slots, void* out, float* part_o, float* part_ml,
                                         unsigned* arrivals, int T, int H, int KV, int hd, float scale, int window,
                                         int max_keys, int out_ld, float softcap, int sink, int keep_first,
-                                        const float* sink_values, cudaStream_t stream) {
+                                        const float* sink_values, int chunk, const float* head_gate, int gate_ld,
+                                        cudaStream_t stream) {
   if (T == 0) return 0;
   if (out_ld <= 0) out_ld = H * hd;                      // elements between rows of out (0: dense)
   TLC_REQUIRE(tlc_attention_decode_fused_ok(H, KV, hd), "attention(decode, fused): %d heads, %d key/value heads of size %d are outside the kernel's range", H, KV, hd);
@@ -423,7 +430,7 @@ extern "C" int tlc_attention_decode_fused(const float* qkv, int ld, int q_off, i
 #define TLC_FM_LAUNCH(HDV, CKV, STV)                                                                                   \
   e = launch_fused<HDV, CKV, STV>(grid, passes, stream, qkv, ld, q_off, k_off, v_off, kp, vp, inv_freq, rope_dim, write_kv, \
                                 block_table, max_pages, positions, row_seq, slots, part_o, part_ml, arrivals, op, H, KV, \
-                                scale, window, n_splits, passes, out_ld, softcap, sink, keep_first, sink_values)
+                                scale, window, n_splits, passes, out_ld, softcap, sink, keep_first, sink_values, chunk, head_gate, gate_ld)
   if (hd == 64) TLC_FM_LAUNCH(64, 32, 4);
   else if (hd == 128) TLC_FM_LAUNCH(128, 32, 2);
   else TLC_FM_LAUNCH(256, 16, 2);

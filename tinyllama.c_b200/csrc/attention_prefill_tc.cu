@@ -76,8 +76,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ start_pos, __nv_bfloat16* __restrict__ out, int n_seqs, int n_tiles, int H,
                             int KV, float scale_log2, int window, int out_ld, int n_split, float* __restrict__ part_o,
                             float* __restrict__ part_ml, float cap_in, float cap_out, int sink, int keep_first,
-                            const float* __restrict__ sink_values, ErrWords* err) {
-  tlc_pdl(out);
+                            const float* __restrict__ sink_values, int chunk, const float* __restrict__ head_gate, int gate_ld,
+                            ErrWords* err) {
+  tlc_pdl(out, head_gate);
   using L_ = FaSmem<HD>;
   constexpr int TCOLS = HD == 128 ? 512 : 256;            // the groups' scores at 0 and 64, their outputs at 128 and 128 + hd
   extern __shared__ uint8_t fa_raw[];
@@ -157,10 +158,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   const int rows = min(BM, n_new - i0);
   const int p0 = start_pos[b] + i0;                       // position of the block's first row
   const int tile_hi_all = (p0 + rows - 1) / BN;
-  const int tile_lo_all = window > 0 ? max(0, p0 + 1 - window) / BN : 0;
+  const int tile_lo_all = tlc_first_key(p0, window, chunk) / BN;
+  const int last_lo = tlc_first_key(p0 + rows - 1, window, chunk);       // key tiles from here on need no lower bound
   // with a window, the key tiles that hold the sequence's first keep_first keys stay visible: those of them that lie in
   // front of the window come first in the item's list of key tiles, then the window's
-  const int n_kept = (window > 0 && keep_first > 0) ? min((keep_first + BN - 1) / BN, tile_lo_all) : 0;
+  const int n_kept = keep_first > 0 ? min((keep_first + BN - 1) / BN, tile_lo_all) : 0;
   const int n_all = n_kept + tile_hi_all - tile_lo_all + 1;
   const int per_range = (n_all + n_split - 1) / n_split;                             // key tiles of a range, rounded up
   const int list_lo = key_range * per_range;
@@ -246,6 +248,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int wg = warp >> 2, quarter = warp & 3, r = 32 * quarter + lane;
     const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
     const int pr = p0 + r;                                // this row's position
+    const int lo_r = tlc_first_key(pr, window, chunk);    // and the first key it sees
     const uint32_t s_at = tmem + lanes + (uint32_t)(wg * BN);
     const uint32_t o_at = tmem + lanes + 128u + (uint32_t)(wg * HD);
     float m_ref = -INFINITY, l = 0.f;                     // the maximum the numerators refer to (scaled, log2), the sum
@@ -271,11 +274,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
       }
       const int kbase = tile_of(j) * BN;
-      if (window > 0 || kbase + BN - 1 > p0) {
+      if (kbase < last_lo || kbase + BN - 1 > p0) {
 #pragma unroll
         for (int c = 0; c < 64; c++) {
           const int kp = kbase + c;
-          if (!(kp <= pr && (window <= 0 || kp > pr - window || kp < keep_first))) sr[c] = 0xff800000u;     // -inf
+          if (!(kp <= pr && (kp >= lo_r || kp < keep_first))) sr[c] = 0xff800000u;     // -inf
         }
       }
       float mx = -INFINITY;
@@ -340,7 +343,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const float m_all = with_sink ? fmaxf(fmaxf(m0, m1), sv) : fmaxf(m0, m1);
     const float w0 = m0 == -INFINITY ? 0.f : ex2_quick(m0 - m_all), w1 = m1 == -INFINITY ? 0.f : ex2_quick(m1 - m_all);
     const float l_all = xch[NG * BM + r] * w0 + xch[(NG + 1) * BM + r] * w1 + (with_sink ? ex2_quick(sv - m_all) : 0.f);
-    const float inv = whole ? 1.0f / l_all : 1.0f;
+    const float inv = whole ? tlc_head_gate(r < rows ? head_gate : nullptr, gate_ld, t0 + i0 + r, h) / l_all : 1.0f;
     const float f0 = w0 * inv, f1 = w1 * inv;
     const bool has0 = n > 0, has1 = n > 1;                // the group had a tile at all (else its accumulator was never written)
     const size_t part_at = whole ? 0 : (((size_t)(t0 + i0 + r) * H + h) * n_split + key_range);
@@ -394,8 +397,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 constexpr int TC_MAX_SPLIT = 8;
 __global__ void __launch_bounds__(128)
 attention_tc_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out,
-                          int H, int hd, int n_split, int out_ld, int sink, const float* __restrict__ sink_values) {
-  tlc_pdl(part_o, part_ml, out);
+                          int H, int hd, int n_split, int out_ld, int sink, const float* __restrict__ sink_values,
+                          const float* __restrict__ head_gate, int gate_ld) {
+  tlc_pdl(part_o, part_ml, out, head_gate);
   const int t = blockIdx.x, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (h >= H) return;
   const size_t at = ((size_t)t * H + h) * n_split;
@@ -414,7 +418,7 @@ attention_tc_merge_kernel(const float* __restrict__ part_o, const float* __restr
     w[z] = lz[z] > 0.f ? exp2f(mz[z] - m) : 0.f;
     l += lz[z] * w[z];
   }
-  const float inv = 1.0f / l;
+  const float inv = tlc_head_gate(head_gate, gate_ld, t, h) / l;
   for (int d = lane * 4; d < hd; d += 128) {
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
@@ -456,7 +460,7 @@ int run(const __nv_bfloat16* q, const __nv_bfloat16* k_pages, const __nv_bfloat1
         const int* block_table, int max_pages, const int* cu_seqlens, const int* slots, const int* start_pos,
         __nv_bfloat16* out, int n_seqs, int n_tiles_bound, int H, int KV, float scale, int window,
         int p_max, int T, int out_ld, int max_blocks, int n_split, float* part_o, float* part_ml, float softcap, int sink,
-        int keep_first, const float* sink_values, cudaStream_t stream) {
+        int keep_first, const float* sink_values, int chunk, const float* head_gate, int gate_ld, cudaStream_t stream) {
   static bool configured = false;
   const int smem = FaSmem<HD>::total(p_max);
   TLC_REQUIRE(smem <= 220 * 1024, "attention(prefill, tcgen05): %d key tiles need %d bytes of shared memory", p_max, smem);
@@ -474,11 +478,12 @@ int run(const __nv_bfloat16* q, const __nv_bfloat16* k_pages, const __nv_bfloat1
   tlc_launch(attention_prefill_tc_kernel<HD>, dim3(blocks), dim3(THREADS), (size_t)smem, stream, mq, mk, mv,
              block_table, max_pages, cu_seqlens, slots, start_pos, out, n_seqs, n_tiles_bound, H, KV, scale * 1.4426950408889634f,
              window, out_ld, n_split, part_o, part_ml, softcap > 0.f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.f,
-             softcap > 0.f ? softcap / scale : 0.f, sink, keep_first, sink_values, tlc_error_words());
+             softcap > 0.f ? softcap / scale : 0.f, sink, keep_first, sink_values, chunk, head_gate, gate_ld,
+             tlc_error_words());
   TLC_CHECK_LAUNCH("attention(prefill, tcgen05)");
   if (n_split > 1) {
     tlc_launch(attention_tc_merge_kernel, dim3(T, (H + 3) / 4), dim3(128), 0, stream, (const float*)part_o, (const float*)part_ml, out, H,
-               HD, n_split, out_ld, sink, sink_values);
+               HD, n_split, out_ld, sink, sink_values, head_gate, gate_ld);
     TLC_CHECK_LAUNCH("attention(prefill, tcgen05, merge)");
   }
   return 0;
@@ -512,13 +517,16 @@ extern "C" int tlc_attention_prefill_tc_ok(int dtype, int hd, int H, int KV) {
 // (32-bit) hold the ranges' results until a second kernel has added them up.
 // softcap > 0: score <- softcap * tanh(score / softcap) after the scale (scale != 0 then); sink: one more term of
 // score 0 in the softmax's denominator, which carries no value (sink_values not NULL: of score sink_values[head]).
-// keep_first > 0 with a window: the sequence's first keep_first keys stay visible.
+// keep_first > 0 with a window: the sequence's first keep_first keys stay visible.  chunk > 0: a row sees the keys of its
+// own chunk of that many positions.  head_gate [T, H] float (rows of gate_ld values, NULL: none): a head's result is
+// multiplied by the sigmoid of its number.
 extern "C" int tlc_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pages, int n_pages,
                                         const int* block_table, int max_pages, const int* cu_seqlens, const int* slots,
                                         const int* start_pos, void* out, int n_seqs, int n_tiles_bound, int H, int KV,
                                         int hd, float scale, int window, int max_keys, int T, int out_ld, int max_blocks,
                                         int n_split, float* part_o, float* part_ml, float softcap, int sink, int keep_first,
-                                        const float* sink_values, cudaStream_t stream) {
+                                        const float* sink_values, int chunk, const float* head_gate, int gate_ld,
+                                        cudaStream_t stream) {
   if (n_seqs == 0 || n_tiles_bound == 0 || T == 0) return 0;
   if (out_ld <= 0) out_ld = H * hd;
   TLC_REQUIRE(tlc_attention_prefill_tc_ok(TLC_BF16, hd, H, KV), "attention(prefill, tcgen05): %d heads, %d key/value heads of size %d are not built", H, KV, hd);
@@ -534,7 +542,7 @@ extern "C" int tlc_attention_prefill_tc(const void* q, const void* k_pages, cons
   const __nv_bfloat16 *qp = (const __nv_bfloat16*)q, *kp = (const __nv_bfloat16*)k_pages, *vp = (const __nv_bfloat16*)v_pages;
   if (hd == 64)
     return run<64>(qp, kp, vp, rows, block_table, max_pages, cu_seqlens, slots, start_pos, (__nv_bfloat16*)out,
-                   n_seqs, n_tiles_bound, H, KV, scale, window, p_max, T, out_ld, max_blocks, n_split, part_o, part_ml, softcap, sink, keep_first, sink_values, stream);
+                   n_seqs, n_tiles_bound, H, KV, scale, window, p_max, T, out_ld, max_blocks, n_split, part_o, part_ml, softcap, sink, keep_first, sink_values, chunk, head_gate, gate_ld, stream);
   return run<128>(qp, kp, vp, rows, block_table, max_pages, cu_seqlens, slots, start_pos, (__nv_bfloat16*)out,
-                  n_seqs, n_tiles_bound, H, KV, scale, window, p_max, T, out_ld, max_blocks, n_split, part_o, part_ml, softcap, sink, keep_first, sink_values, stream);
+                  n_seqs, n_tiles_bound, H, KV, scale, window, p_max, T, out_ld, max_blocks, n_split, part_o, part_ml, softcap, sink, keep_first, sink_values, chunk, head_gate, gate_ld, stream);
 }

@@ -7,12 +7,13 @@
 
 // part_o [T, H, n_splits, HD], part_ml [T, H, n_splits, 2]; out: rows of out_ld elements, head h at h * HD;
 // sh: the block's dynamic shared memory of smem_floats floats (free by now); NT threads.  All threads of
-// the block call it.  sink: one more split of maximum 0 (or sink_values[head]) and sum 1 that carries no values.
+// the block call it.  head_gate: see tlc_head_gate.  sink: one more split of maximum 0 (or sink_values[head]) and sum 1 that carries no values.
 template <int HD, int NT>
 __device__ __forceinline__ void attention_merge_splits(const float* part_o, const float* part_ml, __nv_bfloat16* out,
                                                        float* sh, int smem_floats, int t, int g, int G, int H,
                                                        int n_splits, int out_ld, int sink = 0,
-                                                       const float* sink_values = nullptr) {
+                                                       const float* sink_values = nullptr, const float* head_gate = nullptr,
+                                                       int gate_ld = 0) {
   const int tid = threadIdx.x, lane = tid & 31, wp = tid >> 5;
   constexpr int NW = NT / 32;
   if (2 * G * n_splits <= smem_floats) {
@@ -36,7 +37,7 @@ __device__ __forceinline__ void attention_merge_splits(const float* part_o, cons
       for (int s = lane; s < n_splits; s += 32) if (e[2 * s + 1] > 0.f) l += e[2 * s + 1] * expf(e[2 * s] - m);
       l = warp_sum(l);
       if (sink) l += expf(sv - m);
-      const float inv = 1.0f / l;
+      const float inv = tlc_head_gate(head_gate, gate_ld, t, g * G + hg) / l;
       for (int s = lane; s < n_splits; s += 32) e[2 * s] = e[2 * s + 1] > 0.f ? expf(e[2 * s] - m) * inv : 0.f;
     }
     __syncthreads();
@@ -72,7 +73,7 @@ __device__ __forceinline__ void attention_merge_splits(const float* part_o, cons
       const float ls = __ldcg(mlh + 2 * s + 1);
       if (ls > 0.f) l += ls * expf(__ldcg(mlh + 2 * s) - m);
     }
-    const float inv = 1.0f / l;
+    const float inv = tlc_head_gate(head_gate, gate_ld, t, g * G + hg) / l;
     for (int d = tid; d < HD; d += NT) {
       float acc = 0.f;
       for (int s = 0; s < n_splits; s++)

@@ -166,6 +166,30 @@ template <bool QUICK> __device__ __forceinline__ float moe_pair_act(int act, int
   }
   return w_out ? y * w : y;
 }
+// The first key that a query at position `pos` sees: with a window of that many keys pos + 1 - window, with chunks of `chunk`
+// positions (counted from the sequence's start) the start of pos's own chunk; 0 turns either off.
+__device__ __forceinline__ int tlc_first_key(int pos, int window, int chunk) {
+  int first = 0;
+  if (window > 0) first = max(0, pos + 1 - window);
+  if (chunk > 0) first = max(first, pos - pos % chunk);
+  return first;
+}
+// What an attention head's result is multiplied by: one number per row and head, the sigmoid of gate [T, H] (rows of gate_ld
+// values; NULL: 1).
+__device__ __forceinline__ float tlc_head_gate(const float* __restrict__ gate, int gate_ld, int t, int h) {
+  return gate ? 1.0f / (1.0f + expf(-gate[(size_t)t * gate_ld + h])) : 1.0f;
+}
+// What a product's epilogue is told: whether it adds into its output, or (in the instantiations that end in a gated
+// activation) that activation's code with the constants of the clamped one.
+struct TlcEpi {
+  int code;
+  float limit, alpha;
+  __host__ __device__ TlcEpi(int c = 0, float l = 0.f, float a = 1.0f) : code(c), limit(l), alpha(a) {}
+  __host__ __device__ operator int() const { return code; }
+};
+template <bool QUICK> __device__ __forceinline__ float glu_epilogue(const TlcEpi& e, float g, float u) {
+  return moe_pair_act<QUICK>(e.code, 1, e.limit, e.alpha, 1.0f, g, u);
+}
 // softplus with the reference's cut-over (cpu_op.c:354-356)
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 

@@ -42,6 +42,48 @@ extern "C" int tlc_embed(const int* tokens, const void* table, int table_dtype, 
   return 0;
 }
 
+// x[t] += table[tokens[t]] * scale: the embedding once more (a pass of a repeated range of layers begins with it).  Four
+// values a thread where rows lie on 16-byte (8-byte) boundaries.
+template <typename TW, int VEC>
+__global__ void __launch_bounds__(256)
+embed_add_kernel(const int* __restrict__ tokens, const TW* __restrict__ table, int D, int V, float scale, float* __restrict__ x) {
+  tlc_pdl(x);
+  const int t = blockIdx.x;
+  int tok = tokens[t];
+  tok = tok < 0 ? 0 : (tok >= V ? V - 1 : tok);
+  const TW* row = table + (size_t)tok * D;
+  float* xr = x + (size_t)t * D;
+  for (int d = threadIdx.x * VEC; d < D; d += blockDim.x * VEC) {
+    if (VEC == 4) {
+      float4 e;
+      if (sizeof(TW) == 2) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(row + d);
+        const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&raw.x), hi = *reinterpret_cast<const __nv_bfloat162*>(&raw.y);
+        e = make_float4(__low2float(lo), __high2float(lo), __low2float(hi), __high2float(hi));
+      } else {
+        e = *reinterpret_cast<const float4*>(row + d);
+      }
+      float4 v = *reinterpret_cast<const float4*>(xr + d);
+      v.x = fmaf(e.x, scale, v.x); v.y = fmaf(e.y, scale, v.y); v.z = fmaf(e.z, scale, v.z); v.w = fmaf(e.w, scale, v.w);
+      *reinterpret_cast<float4*>(xr + d) = v;
+    } else {
+      xr[d] = fmaf(to_f32(row[d]), scale, xr[d]);
+    }
+  }
+}
+
+extern "C" int tlc_embed_add(const int* tokens, const void* table, int table_dtype, int T, int D, int V, float scale, float* x,
+                             cudaStream_t stream) {
+  if (T == 0) return 0;
+  const bool vec = D % 4 == 0 && (uintptr_t)table % 16 == 0 && (uintptr_t)x % 16 == 0;
+  TLC_DISPATCH_DTYPE(table_dtype, TW, {
+    if (vec) tlc_launch(embed_add_kernel<TW, 4>, dim3(T), dim3(256), 0, stream, tokens, (const TW*)table, D, V, scale, x);
+    else tlc_launch(embed_add_kernel<TW, 1>, dim3(T), dim3(256), 0, stream, tokens, (const TW*)table, D, V, scale, x);
+  });
+  TLC_CHECK_LAUNCH("embed_add");
+  return 0;
+}
+
 // ---- RMSNorm of 32-bit rows ----------------------------------------------------------
 // One block per row.  The row stays in registers between the sum of squares and the scaling
 // when it fits (up to RMS_MAX_PER_THREAD values per thread), otherwise it is read twice.

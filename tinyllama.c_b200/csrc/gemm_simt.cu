@@ -16,7 +16,7 @@
 template <typename TA, typename TW, typename TO>
 __global__ void __launch_bounds__(256)
 gemm_tiled_kernel(const TA* __restrict__ a, int lda, const TW* __restrict__ w, int ldw, TO* __restrict__ out, int ldo,
-                  const float* __restrict__ colscale, const float* __restrict__ colbias, int accumulate, int M, int N,
+                  const float* __restrict__ colscale, const float* __restrict__ colbias, TlcEpi accumulate, int M, int N,
                   int K) {
   tlc_pdl(a, out);
   __shared__ float As[BK][BM + 4];
@@ -70,7 +70,7 @@ gemm_tiled_kernel(const TA* __restrict__ a, int lda, const TW* __restrict__ w, i
 template <typename TA, typename TW, typename TO, int MT>
 __global__ void __launch_bounds__(256)
 gemm_skinny_kernel(const TA* __restrict__ a, int lda, const TW* __restrict__ w, int ldw, TO* __restrict__ out, int ldo,
-                   const float* __restrict__ colscale, const float* __restrict__ colbias, int accumulate, int M, int N,
+                   const float* __restrict__ colscale, const float* __restrict__ colbias, TlcEpi accumulate, int M, int N,
                    int K, int m_base) {
   tlc_pdl(a, out);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -104,7 +104,7 @@ template <typename TO, int MT>
 __global__ void __launch_bounds__(256)
 gemm_skinny_bf16x8_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfloat16* __restrict__ w, int ldw,
                           TO* __restrict__ out, int ldo, const float* __restrict__ colscale,
-                          const float* __restrict__ colbias, int accumulate, int M, int N, int K, int m_base) {
+                          const float* __restrict__ colbias, TlcEpi accumulate, int M, int N, int K, int m_base) {
   tlc_pdl(a, out);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n = blockIdx.x * (blockDim.x >> 5) + warp;
@@ -149,7 +149,7 @@ gemm_skinny_bf16x8_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __
 
 template <typename TA, typename TW, typename TO>
 static int launch_simt(const void* a, int lda, const void* w, int ldw, void* out, int ldo, const float* colscale,
-                       const float* colbias, int accumulate, int M, int N, int K, cudaStream_t stream) {
+                       const float* colbias, TlcEpi accumulate, int M, int N, int K, cudaStream_t stream) {
   constexpr int MT = 8;
   if (M <= 16) {
     const bool vec = std::is_same<TA, __nv_bfloat16>::value && std::is_same<TW, __nv_bfloat16>::value && (K % 8 == 0) &&
@@ -217,7 +217,7 @@ template <typename TO, int MG, int U, bool SWIGLU, bool PAIR>
 __global__ void __launch_bounds__(SK_WARPS * 32, ((MG == 1 && U <= 4) || (MG == 2 && U <= 2) || (MG == 4 && U == 1)) ? 2 : 1)
 gemm_skinny_mma_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfloat16* __restrict__ w, int ldw,
                        TO* __restrict__ out, int ldo, const float* __restrict__ colscale,
-                       const float* __restrict__ colbias, int accumulate, int M, int N, int K) {
+                       const float* __restrict__ colbias, TlcEpi accumulate, int M, int N, int K) {
   static_assert(!(PAIR && SWIGLU), "the paired form has no SwiGLU epilogue");
   // The weights do not depend on the previous kernel of the stream, the activations do: when this
   // kernel is launched early (programmatic dependent launch), the first round of weight loads is
@@ -298,7 +298,7 @@ gemm_skinny_mma_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_
         if (nu < N && m < M) {
           if (colscale) { vg *= colscale[ng]; vu *= colscale[nu]; }
           if (colbias) { vg += colbias[ng]; vu += colbias[nu]; }
-          out[(size_t)m * ldo + (n0 >> 1) + (ln >> 2)] = from_f32<TO>(glu_act_of<false>(accumulate, vg) * vu);   // (the activation's code)
+          out[(size_t)m * ldo + (n0 >> 1) + (ln >> 2)] = from_f32<TO>(glu_epilogue<false>(accumulate, vg, vu));   // (the activation's code)
         }
       }
       continue;
@@ -341,7 +341,7 @@ gemm_skinny_mma_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_
 
 template <typename TO, int MG, bool SWIGLU>
 static void launch_skinny_mg(const __nv_bfloat16* a, int lda, const __nv_bfloat16* w, int ldw, TO* out, int ldo,
-                             const float* colscale, const float* colbias, int accumulate, int M, int N, int K,
+                             const float* colscale, const float* colbias, TlcEpi accumulate, int M, int N, int K,
                              cudaStream_t stream) {
   const unsigned blocks = (unsigned)((N + 15) / 16);
   const int n_steps = ((K >> 3) + 3) >> 2;
@@ -384,7 +384,7 @@ static void launch_skinny_mg(const __nv_bfloat16* a, int lda, const __nv_bfloat1
 
 template <typename TO, bool SWIGLU>
 static int launch_skinny_mma(const void* a, int lda, const void* w, int ldw, void* out, int ldo, const float* colscale,
-                             const float* colbias, int accumulate, int M, int N, int K, cudaStream_t stream) {
+                             const float* colbias, TlcEpi accumulate, int M, int N, int K, cudaStream_t stream) {
   const __nv_bfloat16* ap = (const __nv_bfloat16*)a;
   const __nv_bfloat16* wp = (const __nv_bfloat16*)w;
   if (M <= 8) launch_skinny_mg<TO, 1, SWIGLU>(ap, lda, wp, ldw, (TO*)out, ldo, colscale, colbias, accumulate, M, N, K, stream);
@@ -414,8 +414,9 @@ extern "C" int tlc_linear_skinny(const void* a, int lda, const void* w, int ldw,
 extern "C" void tlc_linear_skinny_pairs(int on) { g_skinny_pairs = on; }
 
 extern "C" int tlc_linear_skinny_swiglu(const void* a, int lda, const void* w, int ldw, void* out, int out_dtype, int ldo,
-                                        const float* colscale, const float* colbias, int M, int N, int K, int act,
-                                        cudaStream_t stream) {
+                                        const float* colscale, const float* colbias, int M, int N, int K, int act_code,
+                                        float limit, float alpha, cudaStream_t stream) {
+  const TlcEpi act(act_code, limit, alpha);
   if (out_dtype == TLC_F32)
     return launch_skinny_mma<float, true>(a, lda, w, ldw, out, ldo, colscale, colbias, act, M, N, K, stream);
   if (out_dtype == TLC_BF16)

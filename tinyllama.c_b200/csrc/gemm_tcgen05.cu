@@ -28,10 +28,10 @@
 
 // gemm_tcgen05_few_rows.cu
 int tlc_linear_few_rows_run(const void* a, int lda, const void* w, int ldw, void* out, int out_dtype, int ldo,
-                            const float* colscale, const float* colbias, int accumulate, int M, int N, int K,
+                            const float* colscale, const float* colbias, TlcEpi accumulate, int M, int N, int K,
                             cudaStream_t stream);
 int tlc_linear_few_rows_swiglu(const void* a, int lda, const void* w, int ldw, void* out, int out_dtype, int ldo,
-                               const float* colscale, const float* colbias, int M, int N, int K, int act, cudaStream_t stream);
+                               const float* colscale, const float* colbias, int M, int N, int K, TlcEpi act, cudaStream_t stream);
 
 namespace {
 
@@ -70,7 +70,7 @@ template <typename TO, int BN, int STAGES, bool SWIGLU, bool PAIR>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                     TO* __restrict__ out, int ldo, const float* __restrict__ colscale,
-                    const float* __restrict__ colbias, int accumulate, int M, int N, int K, ErrWords* err,
+                    const float* __restrict__ colbias, TlcEpi accumulate, int M, int N, int K, ErrWords* err,
                     int splits, float* __restrict__ part, unsigned* __restrict__ arrivals,
                     const __grid_constant__ CUtensorMap map_o, int tma_out) {
   // The set-up and the first weight tiles do not depend on the previous kernel of the stream: they go ahead of
@@ -317,7 +317,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
               vg = vg * sc[jg] + sc[BN + jg];
               vu = vu * sc[jg + 8] + sc[BN + jg + 8];
             }
-            o16[f] = glu_act_of<true>(accumulate, vg) * vu;       // (with SWIGLU the argument carries the activation's code)
+            o16[f] = glu_epilogue<true>(accumulate, vg, vu);       // (with SWIGLU the argument carries the activation's code)
           }
           if (m < M) {
             TO* dst = out + (size_t)m * ldo + oc0;
@@ -675,7 +675,7 @@ int pick_splits(int M, int N, int K, int bn) {
 
 template <typename TO, int BN, int STAGES, bool SWIGLU = false>
 int launch(const CUtensorMap& ma, const CUtensorMap& mb, void* out, int ldo, const float* colscale, const float* colbias,
-           int accumulate, int M, int N, int K, cudaStream_t stream) {
+           TlcEpi accumulate, int M, int N, int K, cudaStream_t stream) {
   using S = Smem<BN, STAGES>;
   auto kern = gemm_tcgen05_kernel<TO, BN, STAGES, SWIGLU, false>;
   int splits = SWIGLU ? 1 : pick_splits(M, N, K, BN);
@@ -704,7 +704,7 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mb, void* out, int ldo, con
 // Pairs of blocks on tiles of 256 x 256: a cluster of two per tile, as many pairs as the GPU runs at once.
 template <typename TO, bool SWIGLU = false>
 int launch_pairs(const CUtensorMap& ma, const CUtensorMap& mb, void* out, int ldo, const float* colscale, const float* colbias,
-                 int accumulate, int M, int N, int K, cudaStream_t stream) {
+                 TlcEpi accumulate, int M, int N, int K, cudaStream_t stream) {
   using S = Smem<PAIR_BN, PAIR_STAGES, true>;
   const int tiles = ((N + PAIR_BN - 1) / PAIR_BN) * ((M + 2 * BM - 1) / (2 * BM));
   cudaLaunchConfig_t cfg = {};
@@ -795,15 +795,19 @@ extern "C" int tlc_linear_tcgen05_ok(int a_dtype, int lda, const void* a, int w_
          ((uintptr_t)a % 16 == 0) && ((uintptr_t)w % 16 == 0);
 }
 
-// The fused feed-forward front: out[M, N/2] = act(gate) * up (act: SiLU or the tanh form of GELU; the kernels' SWIGLU
+// The fused feed-forward front: out[M, N/2] = act(gate) * up (act: SiLU, the tanh form of GELU, or the clamped swish, whose result has no
+// plain product: see moe_pair_act; the kernels' SWIGLU
 // instantiations take its code in the argument that is `accumulate` elsewhere), where the rows of w come in groups of
 // 16 (8 gate rows, then their 8 up rows) and gate/up = (a w^T) * colscale + colbias.  Returns 1 if no
 // kernel takes these operands (the caller then runs the product and the activation separately).
 extern "C" int tlc_linear_swiglu(const void* a, int a_dtype, int lda, const void* w, int w_dtype, int ldw, void* out,
                                  int out_dtype, int ldo, const float* colscale, const float* colbias, int M, int N, int K,
-                                 int min_rows_for_tensor_cores, int act, cudaStream_t stream) {
+                                 int min_rows_for_tensor_cores, int act_code, float limit, float alpha,
+                                 cudaStream_t stream) {
   if (M == 0 || N == 0) return 0;
-  TLC_REQUIRE(act == TLC_ACT_SILU || act == TLC_ACT_GELU_TANH, "linear_swiglu: unknown activation %d", act);
+  TLC_REQUIRE(act_code == TLC_ACT_SILU || act_code == TLC_ACT_GELU_TANH || act_code == TLC_ACT_SWISH_CLAMPED,
+              "linear_swiglu: unknown activation %d", act_code);
+  const TlcEpi act(act_code, limit, alpha);
   if (N % 16 != 0 || !tlc_linear_tcgen05_ok(a_dtype, lda, a, w_dtype, ldw, w, K)) return 1;
   TLC_REQUIRE(K > 0 && lda >= K && ldw >= K && ldo >= N / 2, "linear: bad sizes M=%d N=%d K=%d lda=%d ldw=%d ldo=%d", M, N, K,
               lda, ldw, ldo);
@@ -813,7 +817,7 @@ extern "C" int tlc_linear_swiglu(const void* a, int a_dtype, int lda, const void
     return tlc_linear_few_rows_swiglu(a, lda, w, ldw, out, out_dtype, ldo, colscale, colbias, M, N, K, act, stream);
   }
   if (M <= 32 && tlc_linear_skinny_ok(a_dtype, lda, a, w_dtype, ldw, w, M, K))
-    return tlc_linear_skinny_swiglu(a, lda, w, ldw, out, out_dtype, ldo, colscale, colbias, M, N, K, act, stream);
+    return tlc_linear_skinny_swiglu(a, lda, w, ldw, out, out_dtype, ldo, colscale, colbias, M, N, K, act_code, limit, alpha, stream);
   if (M < min_rows_for_tensor_cores) return 1;
   if (int rc = init_once()) return rc;
   CUtensorMap ma, mb;

@@ -54,7 +54,7 @@ template <typename TO, int NB, int STAGES, bool SWIGLU>
 __global__ void __launch_bounds__(FR_THREADS, 2)
 gemm_few_rows_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                      TO* __restrict__ out, int ldo, const float* __restrict__ colscale,
-                     const float* __restrict__ colbias, int accumulate, int M, int N, int K, int split, ErrWords* err) {
+                     const float* __restrict__ colbias, TlcEpi accumulate, int M, int N, int K, int split, ErrWords* err) {
   asm volatile("griddepcontrol.launch_dependents;");
   using S = FrSmem<NB, STAGES>;
   extern __shared__ uint8_t fr_raw[];
@@ -196,7 +196,7 @@ gemm_few_rows_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_con
         v = v * cs + cb;
         if (SWIGLU) {
           v2 = v2 * cs2 + cb2;
-          out[(size_t)m * ldo + (n0 >> 1) + ((row >> 4) << 3) + (row & 7)] = from_f32<TO>(glu_act_of<false>(accumulate, v) * v2);      // (with SWIGLU the argument carries the activation's code)
+          out[(size_t)m * ldo + (n0 >> 1) + ((row >> 4) << 3) + (row & 7)] = from_f32<TO>(glu_epilogue<false>(accumulate, v, v2));      // (with SWIGLU the argument carries the activation's code)
         } else {
           TO* o = out + (size_t)m * ldo + n;
           if (accumulate) v += to_f32(*o);
@@ -225,7 +225,7 @@ int g_max_split[4] = {0, 0, 0, 0};      // [log2 split]: how many clusters of th
 
 template <typename TO, int NB, int STAGES, bool SWIGLU>
 int launch_few(const CUtensorMap& mw, const CUtensorMap& mx, void* out, int ldo, const float* colscale, const float* colbias,
-               int accumulate, int M, int N, int K, int split, cudaStream_t stream) {
+               TlcEpi accumulate, int M, int N, int K, int split, cudaStream_t stream) {
   using S = FrSmem<NB, STAGES>;
   static bool attr_set = false;
   if (!attr_set) {
@@ -274,7 +274,7 @@ int pick_split(int N, int K, int NB, int sms) {
 
 template <bool SWIGLU>
 int run_few(const void* a, int lda, const void* w, int ldw, void* out, int out_dtype, int ldo, const float* colscale,
-            const float* colbias, int accumulate, int M, int N, int K, int force_split, cudaStream_t stream) {
+            const float* colbias, TlcEpi accumulate, int M, int N, int K, int force_split, cudaStream_t stream) {
   static int sms = 0;
   if (sms == 0) { int dev = 0; cudaGetDevice(&dev); cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev); }
   const int NB = M <= 32 ? 32 : M <= 64 ? 64 : 128;
@@ -317,12 +317,12 @@ extern "C" int tlc_linear_few_rows_ok(int a_dtype, int lda, const void* a, int w
 }
 
 int tlc_linear_few_rows_run(const void* a, int lda, const void* w, int ldw, void* out, int out_dtype, int ldo,
-                            const float* colscale, const float* colbias, int accumulate, int M, int N, int K,
+                            const float* colscale, const float* colbias, TlcEpi accumulate, int M, int N, int K,
                             cudaStream_t stream) {
   return run_few<false>(a, lda, w, ldw, out, out_dtype, ldo, colscale, colbias, accumulate, M, N, K, g_force_split, stream);
 }
 
 int tlc_linear_few_rows_swiglu(const void* a, int lda, const void* w, int ldw, void* out, int out_dtype, int ldo,
-                               const float* colscale, const float* colbias, int M, int N, int K, int act, cudaStream_t stream) {
+                               const float* colscale, const float* colbias, int M, int N, int K, TlcEpi act, cudaStream_t stream) {
   return run_few<true>(a, lda, w, ldw, out, out_dtype, ldo, colscale, colbias, act, M, N, K, g_force_split, stream);
 }

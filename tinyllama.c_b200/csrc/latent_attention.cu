@@ -12,7 +12,8 @@
 // The softmax has a sink: a per-head logit, used as stored (the score scale does not apply to it), that adds a single
 // term to the denominator and nothing to the weighted sum of values.  Scores, softmax statistics, rotation angles, the norm of c and all
 // accumulators are 32-bit.  The rotation is the interleaved one: dimensions (2i, 2i+1) of the first `rot` dimensions
-// turn by position * inv_freq[i]; what lies beyond passes unchanged.
+// turn by position * inv_freq[i] (cosines and sines times `amplitude`); what lies beyond passes unchanged.  A head's
+// result may be multiplied by the sigmoid of one number per row and head (head_gate): an output gate that commutes with V_h.
 #include "common.cuh"
 
 // ---- per row: rotate, norm, store ---------------------------------------------------------------------
@@ -26,7 +27,7 @@ latent_prepare_kernel(const float* __restrict__ qproj, int ldq, int q_off, const
                       const float* __restrict__ inv_freq, int rot, const int* __restrict__ positions,
                       const int* __restrict__ row_seq, const int* __restrict__ slots, const int* __restrict__ block_table,
                       int max_pages, TC* __restrict__ pages, TC* __restrict__ qn, TC* __restrict__ qa, int H, int dn, int r,
-                      int R) {
+                      int R, float amplitude) {
   tlc_pdl(qproj, proj, pages, qn, qa);
   __shared__ float red[33];
   const int t = blockIdx.x;
@@ -47,6 +48,8 @@ latent_prepare_kernel(const float* __restrict__ qproj, int ldq, int q_off, const
     if (j < half) {
       float sn, cs;
       sincosf(fpos * inv_freq[j], &sn, &cs);
+      sn *= amplitude;
+      cs *= amplitude;
       const float u = src[2 * j], v = src[2 * j + 1];
       dst[2 * j] = from_f32<TC>(u * cs - v * sn);
       dst[2 * j + 1] = from_f32<TC>(v * cs + u * sn);
@@ -69,6 +72,8 @@ latent_prepare_kernel(const float* __restrict__ qproj, int ldq, int q_off, const
     if (j < half) {
       float sn, cs;
       sincosf(fpos * inv_freq[j], &sn, &cs);
+      sn *= amplitude;
+      cs *= amplitude;
       const float u = src[2 * j], v = src[2 * j + 1];
       row[R + 2 * j] = from_f32<TC>(u * cs - v * sn);
       row[R + 2 * j + 1] = from_f32<TC>(v * cs + u * sn);
@@ -83,13 +88,13 @@ extern "C" int tlc_latent_prepare(const float* qproj, int ldq, int q_off, const 
                                   float eps,
                                   const float* inv_freq, int rot, const int* positions, const int* row_seq, const int* slots,
                                   const int* block_table, int max_pages, void* pages, void* qn, void* qa, int dtype, int T, int H,
-                                  int dn, int r, int R, cudaStream_t stream) {
+                                  int dn, int r, int R, float amplitude, cudaStream_t stream) {
   if (T == 0) return 0;
   TLC_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= r, "latent_prepare: %d rotated dimensions of %d", rot, r);
   const int nt = T < 256 ? 512 : 128;                       // few rows: more threads a row
   TLC_DISPATCH_DTYPE(dtype, TC, tlc_launch(latent_prepare_kernel<TC>, dim3(T), dim3(nt), 0, stream, qproj, ldq, q_off, proj, ld, dkv_off, cw, eps,
                                            inv_freq, rot, positions, row_seq, slots, block_table, max_pages, (TC*)pages, (TC*)qn,
-                                           (TC*)qa, H, dn, r, R));
+                                           (TC*)qa, H, dn, r, R, amplitude));
   TLC_CHECK_LAUNCH("latent_prepare");
   return 0;
 }
@@ -103,8 +108,8 @@ __global__ void __launch_bounds__(128)
 latent_attention_warp_kernel(const TC* __restrict__ qa, const TC* __restrict__ pages, const float* __restrict__ sink,
                              const int* __restrict__ block_table, int max_pages, const int* __restrict__ positions,
                              const int* __restrict__ row_seq, const int* __restrict__ slots, TC* __restrict__ out, int H, int R,
-                             int r, float scale, int window) {
-  tlc_pdl(qa, pages, out);
+                             int r, float scale, int window, const float* __restrict__ head_gate, int gate_ld) {
+  tlc_pdl(qa, pages, out, head_gate);
   extern __shared__ float sh[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x, h = blockIdx.y * 4 + warp;
@@ -150,7 +155,7 @@ latent_attention_warp_kernel(const TC* __restrict__ qa, const TC* __restrict__ p
     }
     m = m_new;
   }
-  const float inv = 1.0f / l;
+  const float inv = tlc_head_gate(head_gate, gate_ld, t, h) / l;
   TC* o = out + ((size_t)t * H + h) * R;
 #pragma unroll
   for (int i = 0; i < LAT_MAXV; i++) {
@@ -161,7 +166,8 @@ latent_attention_warp_kernel(const TC* __restrict__ qa, const TC* __restrict__ p
 
 extern "C" int tlc_latent_attention(const void* qa, const void* pages, int dtype, const float* sink, const int* block_table,
                                     int max_pages, const int* positions, const int* row_seq, const int* slots, void* out, int T,
-                                    int H, int R, int r, float scale, int window, cudaStream_t stream) {
+                                    int H, int R, int r, float scale, int window, const float* head_gate, int gate_ld,
+                                    cudaStream_t stream) {
   if (T == 0) return 0;
   TLC_REQUIRE(R >= 1 && R <= 32 * LAT_MAXV, "latent_attention: a latent of %d values exceeds the kernel's limit of %d", R, 32 * LAT_MAXV);
   const size_t smem = (size_t)4 * (R + r) * sizeof(float);
@@ -169,7 +175,7 @@ extern "C" int tlc_latent_attention(const void* qa, const void* pages, int dtype
   dim3 grid(T, (H + 3) / 4);
   TLC_DISPATCH_DTYPE(dtype, TC, tlc_launch(latent_attention_warp_kernel<TC>, grid, dim3(128), smem, stream, (const TC*)qa,
                                            (const TC*)pages, sink, block_table, max_pages, positions, row_seq, slots, (TC*)out, H, R, r,
-                                           scale, window));
+                                           scale, window, head_gate, gate_ld));
   TLC_CHECK_LAUNCH("latent_attention");
   return 0;
 }
@@ -269,8 +275,9 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ qa, const __nv_bflo
                            const float* __restrict__ sink, const int* __restrict__ block_table, int max_pages,
                            const int* __restrict__ cu_seqlens, const int* __restrict__ slots, const int* __restrict__ start_pos,
                            __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int B, int H,
-                           int HP, int R, int r, float scale, int n_split, int n_tiles, int window) {
-  tlc_pdl(qa, pages, out, part_o, part_ml);
+                           int HP, int R, int r, float scale, int n_split, int n_tiles, int window,
+                           const float* __restrict__ head_gate, int gate_ld) {
+  tlc_pdl(qa, pages, out, part_o, part_ml, head_gate);
   constexpr int LTM = NWARP * 16, NT = NWARP * 32;
   extern __shared__ __align__(16) unsigned char lt_smem[];
   const int aw = R + r, ldsm = aw + 8;                    // padded row: ldmatrix rows land in different banks
@@ -450,7 +457,7 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ qa, const __nv_bflo
       const float sk = sink ? sink[h] : -INFINITY;         // no sink: nothing joins the denominator
       const float mf = fmaxf(m_run[e], sk);
       const float w = exp2f((m_run[e] - mf) * LOG2E);
-      const float inv = w / (l_run[e] * w + exp2f((sk - mf) * LOG2E));
+      const float inv = w * tlc_head_gate(head_gate, gate_ld, t0 + rl, h) / (l_run[e] * w + exp2f((sk - mf) * LOG2E));
       __nv_bfloat16* po = out + th * R;
 #pragma unroll
       for (int i = 0; i < MAXNV; i++)
@@ -467,8 +474,9 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ qa, const __nv_bflo
 // thread per output column, all ranges' loads of a column in flight together.
 __global__ void __launch_bounds__(128)
 latent_attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const float* __restrict__ sink,
-                              __nv_bfloat16* __restrict__ out, int H, int R, int n_split) {
-  tlc_pdl(part_o, part_ml, out);
+                              __nv_bfloat16* __restrict__ out, int H, int R, int n_split,
+                              const float* __restrict__ head_gate, int gate_ld) {
+  tlc_pdl(part_o, part_ml, out, head_gate);
   __shared__ float wsh[64];
   const int th = blockIdx.x;
   const float sk = sink ? sink[th % H] : -INFINITY;
@@ -477,7 +485,7 @@ latent_attention_merge_kernel(const float* __restrict__ part_o, const float* __r
   for (int s = 0; s < n_split; s++) mf = fmaxf(mf, ml[2 * s]);
   float den = expf(sk - mf);
   for (int s = 0; s < n_split; s++) den += ml[2 * s + 1] * expf(ml[2 * s] - mf);     // an empty range: sum 0, exp(-inf) = 0
-  const float inv = 1.0f / den;
+  const float inv = tlc_head_gate(head_gate, gate_ld, th / H, th % H) / den;
   if (threadIdx.x < n_split) wsh[threadIdx.x] = expf(ml[2 * threadIdx.x] - mf) * inv;
   __syncthreads();
   for (int d = threadIdx.x; d < R; d += blockDim.x) {
@@ -522,7 +530,7 @@ extern "C" int tlc_latent_attention_tc_splits(int n_tiles, int max_keys) {
 extern "C" int tlc_latent_attention_tc(const void* qa, const void* pages, const float* sink, const int* block_table, int max_pages,
                                        const int* cu_seqlens, const int* slots, const int* start_pos, void* out, float* part_o,
                                        float* part_ml, int B, int T, int tile_pairs, int n_tiles, int H, int R, int r, float scale,
-                                       int n_split, int window, cudaStream_t stream) {
+                                       int n_split, int window, const float* head_gate, int gate_ld, cudaStream_t stream) {
   if (T == 0) return 0;
   TLC_REQUIRE(tlc_latent_attention_tc_ok(TLC_BF16, H, R, r), "latent_attention_tc: sizes H=%d R=%d r=%d are not built", H, R, r);
   TLC_REQUIRE(n_split >= 1 && n_split <= 64 && (n_split == 1 || (part_o && part_ml)), "latent_attention_tc: %d key ranges (1..64; more than one needs scratch)", n_split);
@@ -543,14 +551,14 @@ extern "C" int tlc_latent_attention_tc(const void* qa, const void* pages, const 
   typedef const __nv_bfloat16* BP;
 #define LT_LAUNCH(NV, NW)                                                                                                      \
   tlc_launch(latent_attention_tc_kernel<NV, NW>, grid, dim3(NW * 32), smem, stream, (BP)qa, (BP)pages, sink, block_table, max_pages, \
-             cu_seqlens, slots, start_pos, (__nv_bfloat16*)out, part_o, part_ml, B, H, HP, R, r, scale, n_split, n_tiles, window)
+             cu_seqlens, slots, start_pos, (__nv_bfloat16*)out, part_o, part_ml, B, H, HP, R, r, scale, n_split, n_tiles, window, head_gate, gate_ld)
   if (tile_pairs == 128) { if (R <= 128) LT_LAUNCH(8, 8); else LT_LAUNCH(16, 8); }
   else { if (R <= 128) LT_LAUNCH(8, 4); else LT_LAUNCH(16, 4); }
 #undef LT_LAUNCH
   TLC_CHECK_LAUNCH("latent_attention_tc");
   if (n_split > 1) {
     tlc_launch(latent_attention_merge_kernel, dim3(T * H), dim3(128), 0, stream, (const float*)part_o, (const float*)part_ml, sink,
-               (__nv_bfloat16*)out, H, R, n_split);
+               (__nv_bfloat16*)out, H, R, n_split, head_gate, gate_ld);
     TLC_CHECK_LAUNCH("latent_attention_merge");
   }
   return 0;

@@ -4,7 +4,8 @@
 // the largest scores (the lowest index wins a tie); its weights are the chosen scores as they are.  The kernel also
 // sorts the (token, choice) pairs by expert -- counts, offsets, and for every expert the list of its pairs -- so that
 // each expert's rows form one contiguous range of a permutation; nothing goes through the host, so the same launches
-// serve any routing (and a captured graph).
+// serve any routing (and a captured graph).  tlc_moe_route_table needs no logits: a table gives every token id its experts,
+// all of one weight.
 //
 // Experts (tlc_moe_gate_up, tlc_moe_down): an expert is fed the token scaled by its weight, expert(w h); gate and up are
 // linear, so W (w h) = w (W h) and the epilogue of the first product applies w in 32 bits: act(w g) * (w u).  The
@@ -90,18 +91,43 @@ moe_topk_kernel(const float* __restrict__ logits, int ld, int T, int E, int top,
   }
 }
 
+// What the sort is told instead of ids where a table routes: a token's experts are the row of `table` [V, top] that its id
+// names, each with the same weight; the kernel then writes ids and weights itself.
+struct MoeTable {
+  const int* tokens;
+  const int* table;
+  int V, top;
+  float weight;
+  int* ids;
+  float* wts;
+};
+
 // One block sorts the pairs by expert: counts, offsets (and every expert's first tile of `tm` sorted rows), then the
 // list order [T*top]: pair index (t * top + k) of every sorted position.
 __global__ void __launch_bounds__(1024)
-moe_sort_kernel(const int* __restrict__ ids, int n_pairs, int E, int E_tiled, int tm, int* __restrict__ order,
-                int* __restrict__ offsets, int* __restrict__ tile_off) {
-  tlc_pdl(ids, order, offsets, tile_off);
+moe_sort_kernel(const int* ids, int n_pairs, int E, int E_tiled, int tm, int* __restrict__ order,
+                int* __restrict__ offsets, int* __restrict__ tile_off, MoeTable by_table) {
+  tlc_pdl(ids, order, offsets, tile_off, by_table.ids, by_table.wts);
   extern __shared__ int shi[];
   int* count = shi;            // [E]
   int* cursor = shi + E;       // [E]
   for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
   __syncthreads();
-  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) atomicAdd(&count[ids[i]], 1);
+  if (by_table.table) {
+    ids = by_table.ids;
+    for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
+      const int t = i / by_table.top;
+      int tok = by_table.tokens[t];
+      tok = tok < 0 ? 0 : (tok >= by_table.V ? by_table.V - 1 : tok);
+      int e = by_table.table[(size_t)tok * by_table.top + (i - t * by_table.top)];
+      e = e < 0 ? 0 : (e >= E ? E - 1 : e);             // (the host checks the table; never index out of bounds)
+      by_table.ids[i] = e;                              // (read again below by this thread only)
+      by_table.wts[i] = by_table.weight;
+      atomicAdd(&count[e], 1);
+    }
+  } else {
+    for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) atomicAdd(&count[ids[i]], 1);
+  }
   __syncthreads();
   if (threadIdx.x == 0) {
     int o = 0, tiles = 0;
@@ -130,8 +156,19 @@ extern "C" int tlc_moe_route(const float* logits, int ld, int T, int E, int top,
   tlc_launch(moe_topk_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, logits, ld, T, E, top, mode, choice_bias, ids, wts, sum_to);
   TLC_CHECK_LAUNCH("moe_topk");
   tlc_launch(moe_sort_kernel, dim3(1), dim3(1024), (size_t)2 * E * sizeof(int), stream, (const int*)ids, T * top, E, E - n_identity, tile_rows,
-             order, offsets, tile_off);
+             order, offsets, tile_off, MoeTable{nullptr, nullptr, 0, 1, 0.f, nullptr, nullptr});
   TLC_CHECK_LAUNCH("moe_sort");
+  return 0;
+}
+
+extern "C" int tlc_moe_route_table(const int* tokens, const int* table, int T, int V, int E, int top, float weight, int* ids, float* wts,
+                                   int* order, int* offsets, int* tile_off, int tile_rows, cudaStream_t stream) {
+  if (T == 0) return 0;
+  TLC_REQUIRE(tile_rows >= 1, "moe_route_table: tiles of %d rows", tile_rows);
+  TLC_REQUIRE(E >= 1 && top >= 1 && top <= E && E <= 4096 && V >= 1, "moe_route_table: %d experts, %d chosen, %d token ids", E, top, V);
+  tlc_launch(moe_sort_kernel, dim3(1), dim3(1024), (size_t)2 * E * sizeof(int), stream, (const int*)nullptr, T * top, E, E, tile_rows,
+             order, offsets, tile_off, MoeTable{tokens, table, V, top, weight, ids, wts});
+  TLC_CHECK_LAUNCH("moe_route_table");
   return 0;
 }
 

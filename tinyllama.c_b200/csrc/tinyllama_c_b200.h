@@ -70,6 +70,9 @@ int tlc_selftest_bounded_wait(cudaStream_t stream);
  * cache contents of earlier steps ahead of their own dependency wait. */
 int tlc_embed(const int* tokens, const void* table, int table_dtype, int T, int D, int V, float scale,
               float* out, cudaStream_t stream);
+/* x[t] += table[tokens[t]] * scale; x float [T, D] (an ordinary kernel of a step, not its first). */
+int tlc_embed_add(const int* tokens, const void* table, int table_dtype, int T, int D, int V, float scale, float* x,
+                  cudaStream_t stream);
 /* out[r] = x[rows ? rows[r] : r] / sqrt(mean(x^2) + eps) * w;  x float, rows of D values x_ld apart (a range of the
  * columns of a wider matrix will do); out [R, D] of out_dtype. */
 int tlc_rmsnorm(const float* x, int x_ld, const int* rows, const float* w, float eps, int R, int D, void* out,
@@ -137,11 +140,12 @@ int tlc_linear(const void* a, int a_dtype, int lda, const void* w, int w_dtype, 
                int out_dtype, int ldo, const float* colscale, const float* colbias, int accumulate, int M,
                int N, int K, int min_rows_for_tensor_cores, cudaStream_t stream);
 /* out[M, N/2] = act(gate) * up where the rows of w come in groups of 16 (8 gate rows, their 8 up rows); act is
- * TLC_ACT_SILU or TLC_ACT_GELU_TANH.  Returns 1 when no fused kernel takes the operands (run tlc_linear and tlc_glu
+ * TLC_ACT_SILU, TLC_ACT_GELU_TANH, or TLC_ACT_SWISH_CLAMPED with its limit and alpha (its result in place of act(gate) * up).
+ * Returns 1 when no fused kernel takes the operands (run tlc_linear and tlc_glu
  * instead). */
 int tlc_linear_swiglu(const void* a, int a_dtype, int lda, const void* w, int w_dtype, int ldw, void* out,
                       int out_dtype, int ldo, const float* colscale, const float* colbias, int M, int N, int K,
-                      int min_rows_for_tensor_cores, int act, cudaStream_t stream);
+                      int min_rows_for_tensor_cores, int act, float limit, float alpha, cudaStream_t stream);
 int tlc_linear_simt(const void* a, int a_dtype, int lda, const void* w, int w_dtype, int ldw, void* out,
                     int out_dtype, int ldo, const float* colscale, const float* colbias, int accumulate,
                     int M, int N, int K, cudaStream_t stream);
@@ -159,7 +163,7 @@ int tlc_linear_skinny(const void* a, int lda, const void* w, int ldw, void* out,
                       cudaStream_t stream);
 int tlc_linear_skinny_swiglu(const void* a, int lda, const void* w, int ldw, void* out, int out_dtype, int ldo,
                              const float* colscale, const float* colbias, int M, int N, int K, int act,
-                             cudaStream_t stream);
+                             float limit, float alpha, cudaStream_t stream);
 int tlc_linear_tcgen05_ok(int a_dtype, int lda, const void* a, int w_dtype, int ldw, const void* w, int K);
 /* Test hooks: force the tile width (0, 64, 128, 256) / how many blocks share a tile's K-steps (0 = choose). */
 void tlc_linear_tile_override(int bn);
@@ -181,21 +185,25 @@ int tlc_rope_kv_store(const void* qkv, int in_dtype, int dtype, int ld, int q_of
  * `window`); any sizes, both element types; a warp per (row, head).  softcap > 0: score <- softcap * tanh(score /
  * softcap) after the scale; sink: one more term of score 0 in the softmax's denominator, which carries no value
  * (sink_values not NULL: of score sink_values[head], not scaled).  keep_first > 0 with a window: the first keep_first keys
- * of the sequence stay visible to every query at their own positions. */
+ * of the sequence stay visible to every query at their own positions.  chunk > 0: a row sees the keys of its own chunk of that
+ * many positions (counted from the sequence's start) only.  head_gate (NULL: none; float [T, H], rows gate_ld apart): head h of
+ * row t's result is multiplied by sigmoid(head_gate[t, h]). */
 int tlc_attention(const void* q, int dtype, const void* k_pages, const void* v_pages, const int* block_table,
                   int max_pages, const int* positions, const int* row_seq, const int* slots, void* out, int T,
                   int H, int KV, int hd, float scale, int window, int out_ld, float softcap, int sink, int keep_first,
-                  const float* sink_values, cudaStream_t stream);
+                  const float* sink_values, int chunk, const float* head_gate, int gate_ld, cudaStream_t stream);
 /* Single-token rows: keys split across blocks of 128, partial results in part_o [T, H, splits, hd] and
- * part_ml [T, H, splits, 2], then merged. */
+ * part_ml [T, H, splits, 2], then merged.  max_keys: the longest sequence, or with a window or chunks (and keep_first 0) their
+ * size + 63 where that is less. */
 int tlc_attention_decode(const void* q, int dtype, const void* k_pages, const void* v_pages,
                          const int* block_table, int max_pages, const int* positions, const int* row_seq,
                          const int* slots, void* out, float* part_o, float* part_ml, int T, int H, int KV,
                          int hd, float scale, int window, int max_keys, int out_ld, float softcap, int sink,
-                         int keep_first, const float* sink_values, cudaStream_t stream);
+                         int keep_first, const float* sink_values, int chunk, const float* head_gate, int gate_ld,
+                         cudaStream_t stream);
 /* Single-token rows of a bfloat16 cache in one kernel: rotation of q and the new key, store of the new
  * K/V row, scores and outputs on the tensor cores, merge of the splits by the last block to arrive
- * (arrivals: zeroed counters, at least T*KV, back at zero afterwards). */
+ * (arrivals: zeroed counters, at least T*KV, back at zero afterwards).  max_keys, chunk and head_gate as above. */
 int tlc_attention_decode_fused_ok(int H, int KV, int hd);
 int tlc_attention_decode_fused_passes(int passes);
 int tlc_attention_decode_fused(const float* qkv, int ld, int q_off, int k_off, int v_off, void* k_pages,
@@ -204,7 +212,7 @@ int tlc_attention_decode_fused(const float* qkv, int ld, int q_off, int k_off, i
                                const int* slots, void* out, float* part_o, float* part_ml, unsigned* arrivals,
                                int T, int H, int KV, int hd, float scale, int window, int max_keys, int out_ld,
                                float softcap, int sink, int keep_first,
-                               const float* sink_values, cudaStream_t stream);
+                               const float* sink_values, int chunk, const float* head_gate, int gate_ld, cudaStream_t stream);
 /* Prompt rows (consecutive positions from start_pos) of a bfloat16 cache on the tensor cores. */
 int tlc_attention_prefill_ok(int dtype, int hd);
 int tlc_attention_prefill_chunks(int n_tiles_bound, int H, int max_tiles, int* chunk_tiles /* host */);
@@ -216,14 +224,15 @@ int tlc_attention_prefill(const void* q, const void* k_pages, const void* v_page
 
 /* The same on tcgen05.mma (attention_prefill_tc.cu): 128-row tiles, Q and the K and V pages by TMA, scores and
  * output in tensor memory.  n_tiles_bound >= sum_b ceil(n_new_b / 128); n_pages: pages of k_pages / v_pages.
- * Values in pages past a sequence's end must be finite.  softcap, sink, keep_first and sink_values as in tlc_attention. */
+ * Values in pages past a sequence's end must be finite.  softcap, sink, keep_first, sink_values, chunk
+ * and head_gate as in tlc_attention. */
 int tlc_attention_prefill_tc_ok(int dtype, int hd, int H, int KV);
 int tlc_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pages, int n_pages,
                              const int* block_table, int max_pages, const int* cu_seqlens, const int* slots,
                              const int* start_pos, void* out, int n_seqs, int n_tiles_bound, int H, int KV,
                              int hd, float scale, int window, int max_keys, int T, int out_ld, int max_blocks,
                              int n_split, float* part_o, float* part_ml, float softcap, int sink, int keep_first,
-                             const float* sink_values, cudaStream_t stream);
+                             const float* sink_values, int chunk, const float* head_gate, int gate_ld, cudaStream_t stream);
 int tlc_attention_prefill_tc_splits(int n_tiles_bound, int H, int max_keys);   // suggested n_split (1: none)
 
 /* ---- Mamba2 (mamba.cu, mamba_ssd.cu) ----------------------------------------------------------------- */
@@ -271,18 +280,18 @@ int tlc_ssm_scan_ssd(const void* xbc, const float* dt, const float* A, const flo
  * [n_pages, TLC_PAGE, R + r].  tlc_latent_prepare reads a row's projections (float: H heads of (dn | r) query values
  * at q_off of qproj, row stride ldq; R + r down-projected values at dkv_off of proj, row stride ld, or dkv_off < 0 for
  * a layer that reads another layer's rows; the two may be one buffer), writes the unrotated query parts to qn [T, H*dn], the rotated ones (interleaved pairs of the
- * first `rot` dimensions, angle = position * inv_freq[i]) into the last r columns of every head of qa [T, H*(R+r)],
+ * first `rot` dimensions, angle = position * inv_freq[i], cosines and sines times amplitude) into the last r columns of every head of qa [T, H*(R+r)],
  * and the row [rmsnorm(c) * cw | rotated kr] into its page.  qn, qa and pages are of `dtype`. */
 int tlc_latent_prepare(const float* qproj, int ldq, int q_off, const float* proj, int ld, int dkv_off, const float* cw, float eps,
                        const float* inv_freq, int rot, const int* positions, const int* row_seq, const int* slots,
                        const int* block_table, int max_pages, void* pages, void* qn, void* qa, int dtype, int T, int H,
-                       int dn, int r, int R, cudaStream_t stream);
+                       int dn, int r, int R, float amplitude, cudaStream_t stream);
 /* out[t, h, :R] = sum_j p_j c_j over the keys 0..position of the row's sequence, p = softmax of (qa[t, h] . [c_j | kr_j])
  * * scale together with the head's sink (float [H], or NULL for none), which enters the maximum and the denominator
- * only.  window > 0: a row sees only the last `window` keys up to its own position. */
+ * only.  window > 0: a row sees only the last `window` keys up to its own position.  head_gate as in tlc_attention. */
 int tlc_latent_attention(const void* qa, const void* pages, int dtype, const float* sink, const int* block_table,
                          int max_pages, const int* positions, const int* row_seq, const int* slots, void* out, int T,
-                         int H, int R, int r, float scale, int window, cudaStream_t stream);
+                         int H, int R, int r, float scale, int window, const float* head_gate, int gate_ld, cudaStream_t stream);
 /* The same on the tensor cores, for bfloat16 rows with R and R + r multiples of 16 and R <= 256 (tlc_..._ok): a block
  * takes tile_pairs (64 or 128) (row, head) pairs of one sequence and reads every page once, as keys and as values.  Rows of
  * a sequence are consecutive positions from start_pos.  n_tiles: an upper bound of the sum over sequences of
@@ -296,7 +305,7 @@ int tlc_latent_attention_tc_tile(int T, int B, int R, int r);      /* 64 or 128 
 int tlc_latent_attention_tc(const void* qa, const void* pages, const float* sink, const int* block_table, int max_pages,
                             const int* cu_seqlens, const int* slots, const int* start_pos, void* out, float* part_o,
                             float* part_ml, int B, int T, int tile_pairs, int n_tiles, int H, int R, int r, float scale,
-                            int n_split, int window, cudaStream_t stream);
+                            int n_split, int window, const float* head_gate, int gate_ld, cudaStream_t stream);
 /* A product per head: out[t, h, n] = sum_k a[t, h, k] w[h, n, k]; a with row stride lda and head stride a_hs, w
  * [H, N, K] dense, out with row stride ldo and head stride o_hs; 32-bit sums. */
 int tlc_linear_heads(const void* a, int a_dtype, int lda, int a_hs, const void* w, int w_dtype, void* out,
@@ -327,9 +336,10 @@ int tlc_qk_rotate_norm(float* qkv, int ld, int q_off, int k_off, int H, int KV, 
                        const float* k_w, float pre_eps, float amplitude, cudaStream_t stream);
 int tlc_gate_mul(void* x, int dtype, int ldx, const float* gate, int ldg, int n, int T, int act, cudaStream_t stream);
 /* In place on the 32-bit projection: the q_n query columns from q_off, all heads together, are divided by their root mean
- * square (eps inside the root) and multiplied by qw [q_n]; the k_n key columns from k_off likewise with kw [k_n]. */
+ * square (eps inside the root) and multiplied by qw [q_n]; the k_n key columns from k_off likewise with kw [k_n].  q_count,
+ * k_count: how many of the columns the mean is over (padded heads: the other columns are zero, with zero weights). */
 int tlc_qk_whole_norm(float* qkv, int ld, int q_off, int q_n, const float* qw, int k_off, int k_n, const float* kw, float eps,
-                      int T, cudaStream_t stream);
+                      int T, int q_count, int k_count, cudaStream_t stream);
 
 /* ---- gated delta rule (delta_rule.cu) -------------------------------------------------------------------
  * Per head: M <- a M; w = b (v - M^T k); M <- M + k w^T; r = M^T q (a the decay, b the write strength `beta`), with M
@@ -361,6 +371,9 @@ int tlc_delta_rule(const float* qkv, int ld, int q_off, int k_off, int v_off, co
  * multiplied by sum_to. */
 int tlc_moe_route(const float* logits, int ld, int T, int E, int top, int mode, const float* choice_bias, int n_identity,
                   int* ids, float* wts, int* order, int* offsets, int* tile_off, int tile_rows, float sum_to, cudaStream_t stream);
+/* The same without a router: token t's experts are table[tokens[t], :] (int [V, top], distinct), each with weight `weight`. */
+int tlc_moe_route_table(const int* tokens, const int* table, int T, int V, int E, int top, float weight, int* ids, float* wts,
+                        int* order, int* offsets, int* tile_off, int tile_rows, cudaStream_t stream);
 /* y[pair, :D] = wts[pair] * x[token(pair), :D] for every pair with ids[pair] >= E. */
 int tlc_moe_identity(const void* x, int x_dtype, int ldx, const int* ids, const float* wts, int T, int top, int E, int D,
                      float* y, cudaStream_t stream);

@@ -5,3 +5,4 @@ from . import porarax  # noqa: F401  (registers Porarax)
 from . import sogazen  # noqa: F401  (registers Sogazen)
 from . import kimutar  # noqa: F401  (registers Kimutar)
 from . import kefetar  # noqa: F401  (registers Kefetar)
+from . import fobatar  # noqa: F401  (registers Fobatar)

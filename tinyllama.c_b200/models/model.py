@@ -136,8 +136,11 @@ class Model:
                 if run.add is not None:            # a learned row joins the stream before this entry (a pass of a repeated range)
                     ops.add_row(x, self.rows_of[run.add[0]][run.add[1]])
                     ready = False
-                wanted = r + 1 < len(self.schedule) and self.layers[self.schedule[r + 1].layer].reads_stream_copy \
-                    and self.schedule[r + 1].add is None
+                if run.add_embedding:              # or the embedding output does
+                    ops.embed_add(step.tokens, self.embed_table, self.embed_scale, x)
+                    ready = False
+                nxt = self.schedule[r + 1] if r + 1 < len(self.schedule) else None
+                wanted = nxt is not None and self.layers[nxt.layer].reads_stream_copy and nxt.add is None and not nxt.add_embedding
                 ready = self.layers[run.layer].forward(x, step, cache.layer_view(r if run.cache is None else run.cache, run.writes,
                                                                                  run.kv_cache), ready, wanted)
         if want_rows is None or want_rows.numel() == 0:

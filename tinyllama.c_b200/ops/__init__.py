@@ -41,6 +41,7 @@ _SIGNATURES = {
     "tlc_wait_limit_cycles": (_i, [_ll]),
     "tlc_selftest_bounded_wait": (_i, [_vp]),
     "tlc_embed": (_i, [_vp, _vp, _i, _i, _i, _i, _f, _vp, _vp]),
+    "tlc_embed_add": (_i, [_vp, _vp, _i, _i, _i, _i, _f, _vp, _vp]),
     "tlc_rmsnorm": (_i, [_vp, _i, _vp, _vp, _f, _i, _i, _vp, _i, _vp]),
     "tlc_layernorm": (_i, [_vp, _i, _vp, _vp, _vp, _f, _i, _i, _vp, _vp, _i, _vp]),
     "tlc_add_row": (_i, [_vp, _vp, _i, _i, _vp]),
@@ -49,11 +50,11 @@ _SIGNATURES = {
     "tlc_swiglu": (_i, [_vp, _i, _i, _i, _i, _vp, _i, _i, _vp]),
     "tlc_gather_rows": (_i, [_vp, _vp, _i, _i, _vp, _vp]),
     "tlc_linear": (_i, [_vp, _i, _i, _vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp]),
-    "tlc_linear_swiglu": (_i, [_vp, _i, _i, _vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp]),
+    "tlc_linear_swiglu": (_i, [_vp, _i, _i, _vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _f, _f, _vp]),
     "tlc_linear_simt": (_i, [_vp, _i, _i, _vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _vp]),
     "tlc_linear_skinny_ok": (_i, [_i, _i, _vp, _i, _i, _vp, _i, _i]),
     "tlc_linear_skinny": (_i, [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _vp]),
-    "tlc_linear_skinny_swiglu": (_i, [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _vp]),
+    "tlc_linear_skinny_swiglu": (_i, [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _f, _f, _vp]),
     "tlc_linear_tcgen05_ok": (_i, [_i, _i, _vp, _i, _i, _vp, _i]),
     "tlc_linear_tile_override": (None, [_i]),
     "tlc_linear_split_override": (None, [_i]),
@@ -68,20 +69,20 @@ _SIGNATURES = {
     "tlc_linear_pairs": (_i, []),
     "tlc_rope_kv_store": (_i, [_vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i,
                                _i, _i, _vp]),
-    "tlc_attention": (_i, [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _f, _i, _i, _vp, _vp]),
+    "tlc_attention": (_i, [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _f, _i, _i, _vp, _i, _vp, _i, _vp]),
     "tlc_attention_decode": (_i, [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i,
-                                  _i, _f, _i, _i, _vp, _vp]),
+                                  _i, _f, _i, _i, _vp, _i, _vp, _i, _vp]),
     "tlc_attention_decode_fused_ok": (_i, [_i, _i, _i]),
     "tlc_attention_decode_fused_passes": (_i, [_i]),
     "tlc_attention_decode_fused": (_i, [_vp, _i, _i, _i, _i, _vp, _vp, _vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp,
-                                        _vp, _i, _i, _i, _i, _f, _i, _i, _i, _f, _i, _i, _vp, _vp]),
+                                        _vp, _i, _i, _i, _i, _f, _i, _i, _i, _f, _i, _i, _vp, _i, _vp, _i, _vp]),
     "tlc_attention_prefill_ok": (_i, [_i, _i]),
     "tlc_attention_prefill_chunks": (_i, [_i, _i, _i, _vp]),
     "tlc_attention_prefill": (_i, [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _vp,
                                    _vp, _i, _i, _vp]),
     "tlc_attention_prefill_tc_ok": (_i, [_i, _i, _i, _i]),
     "tlc_attention_prefill_tc": (_i, [_vp, _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i,
-                                      _i, _i, _i, _i, _vp, _vp, _f, _i, _i, _vp, _vp]),
+                                      _i, _i, _i, _i, _vp, _vp, _f, _i, _i, _vp, _i, _vp, _i, _vp]),
     "tlc_attention_prefill_tc_splits": (_i, [_i, _i, _i]),
     "tlc_mamba_conv": (_i, [_vp, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i,
                             _i, _i, _i, _i, _i, _i, _vp]),
@@ -98,7 +99,7 @@ _SIGNATURES = {
     "tlc_convert": (_i, [_vp, _i, _i, _i, _vp, _i, _i, _i, _vp]),
     "tlc_softcap": (_i, [_vp, _ll, _f, _vp]),
     "tlc_rmsnorm_mean_add": (_i, [_vp, _i, _vp, _f, _f, _vp, _f, _i, _i, _vp, _i, _vp, _i, _vp]),
-    "tlc_qk_whole_norm": (_i, [_vp, _i, _i, _i, _vp, _i, _i, _vp, _f, _i, _vp]),
+    "tlc_qk_whole_norm": (_i, [_vp, _i, _i, _i, _vp, _i, _i, _vp, _f, _i, _i, _i, _vp]),
     "tlc_shift_mix": (_i, [_vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp]),
     "tlc_wkv_scan": (_i, [_vp, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _vp]),
     "tlc_rmsnorm_conv": (_i, [_vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]),
@@ -114,19 +115,20 @@ _SIGNATURES = {
     "tlc_rmsnorm_shift": (_i, [_vp, _vp, _vp, _f, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp]),
     "tlc_rmsnorm_add": (_i, [_vp, _i, _vp, _vp, _i, _i, _vp, _f, _i, _i, _vp, _i, _vp, _i, _vp]),
     "tlc_latent_prepare": (_i, [_vp, _i, _i, _vp, _i, _i, _vp, _f, _vp, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i,
-                                _i, _i, _vp]),
-    "tlc_latent_attention": (_i, [_vp, _vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _vp]),
+                                _i, _i, _f, _vp]),
+    "tlc_latent_attention": (_i, [_vp, _vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _vp, _i, _vp]),
     "tlc_latent_attention_tc_ok": (_i, [_i, _i, _i, _i]),
     "tlc_latent_attention_tc_splits": (_i, [_i, _i]),
     "tlc_latent_attention_tc_tile": (_i, [_i, _i, _i, _i]),
     "tlc_latent_attention_tc": (_i, [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i,
-                                     _vp]),
+                                     _vp, _i, _vp]),
     "tlc_linear_heads": (_i, [_vp, _i, _i, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]),
     "tlc_grouped_mma_ok": (_i, [_i, _i, _vp, _i, _i, _vp, _i]),
     "tlc_linear_heads_mma": (_i, [_vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]),
     "tlc_moe_experts_mma": (_i, [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp, _i, _i, _i, _f, _f, _vp]),
     "tlc_mingru_scan": (_i, [_vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _vp, _vp]),
     "tlc_moe_route": (_i, [_vp, _i, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _f, _vp]),
+    "tlc_moe_route_table": (_i, [_vp, _vp, _i, _i, _i, _i, _f, _vp, _vp, _vp, _vp, _vp, _i, _vp]),
     "tlc_moe_gate_up": (_i, [_vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _i, _i, _i, _f, _f, _vp]),
     "tlc_qk_rotate_norm": (_i, [_vp, _i, _i, _i, _i, _i, _i, _i, _vp, _i, _i, _f, _vp, _i, _vp, _vp, _f, _f, _vp]),
     "tlc_gate_mul": (_i, [_vp, _i, _i, _vp, _i, _i, _i, _i, _vp]),
@@ -267,6 +269,17 @@ def embed(tokens: torch.Tensor, table: torch.Tensor, scale: float, out: torch.Te
           out.data_ptr(), _stream())
 
 
+def embed_add(tokens: torch.Tensor, table: torch.Tensor, scale: float, x: torch.Tensor) -> None:
+    """x[t] += table[tokens[t]] * scale; x contiguous float32 [T, D]."""
+    _gpu(tokens, table, x)
+    _i32(tokens, "embed tokens")
+    T, (V, D) = tokens.numel(), table.shape
+    if x.dtype != torch.float32 or not x.is_contiguous() or tuple(x.shape) != (T, D) or not table.is_contiguous():
+        raise KernelError("embed_add: x must be contiguous float32 [T, D] and the table contiguous")
+    _call("tlc_embed_add", tokens.data_ptr(), table.data_ptr(), dtype_code(table.dtype), T, D, V, float(scale), x.data_ptr(),
+          _stream())
+
+
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
             rows: Optional[torch.Tensor] = None) -> None:
     """out[r] = rmsnorm(x[rows[r]] or x[r]) * weight; x float32 [*, D] with dense rows (a range of the columns of a
@@ -324,7 +337,7 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleaved: bool = False) 
 
 
 GLU_ACTS = {"silu": 0, "gelu_tanh": 1}
-DENSE_ACTS = dict(GLU_ACTS, swish_clamped=2)       # the clamped swish has no fused product epilogue: product, then glu()
+DENSE_ACTS = dict(GLU_ACTS, swish_clamped=2)
 
 
 def glu(gate_up: torch.Tensor, out: torch.Tensor, act: str = "silu", interleaved: bool = False, limit: float = 0.0,
@@ -335,7 +348,7 @@ def glu(gate_up: torch.Tensor, out: torch.Tensor, act: str = "silu", interleaved
     T, F2 = gate_up.shape
     F = F2 // 2
     if act not in DENSE_ACTS:
-        raise KernelError(f"glu: unknown activation '{act}'; known: {sorted(GLU_ACTS)}")
+        raise KernelError(f"glu: unknown activation '{act}'; known: {sorted(DENSE_ACTS)}")
     if not out.is_contiguous() or tuple(out.shape) != (T, F) or F2 != 2 * F:
         raise KernelError("glu: out must be contiguous [T, F]")
     if interleaved and F % 8:
@@ -539,12 +552,12 @@ def linear_pairs() -> int:
 
 
 def linear_swiglu(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, colscale: Optional[torch.Tensor] = None,
-                  colbias: Optional[torch.Tensor] = None, act: str = "silu") -> None:
+                  colbias: Optional[torch.Tensor] = None, act: str = "silu", limit: float = 0.0, alpha: float = 1.0) -> None:
     """out[M, F] = act(gate) * up with gate | up = (a w^T) * colscale + colbias, the 2F rows of w in
-    groups of 16 (8 gate rows followed by their 8 up rows); act: "silu" or "gelu_tanh".  One kernel where the
+    groups of 16 (8 gate rows followed by their 8 up rows); act, limit and alpha as in glu().  One kernel where the
     operands allow it (bfloat16, 16-byte aligned rows), else the product and the activation one after the other."""
-    if act not in GLU_ACTS:
-        raise KernelError(f"linear_swiglu: unknown activation '{act}'; known: {sorted(GLU_ACTS)}")
+    if act not in DENSE_ACTS:
+        raise KernelError(f"linear_swiglu: unknown activation '{act}'; known: {sorted(DENSE_ACTS)}")
     _gpu(a, w, out, colscale, colbias)
     M, K = a.shape
     N = w.shape[0]
@@ -557,12 +570,12 @@ def linear_swiglu(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, colscale:
     _launches += 1
     rc = lib.tlc_linear_swiglu(a.data_ptr(), dtype_code(a.dtype), _rows(a, "linear input"), w.data_ptr(), dtype_code(w.dtype),
                                _rows(w, "linear weight"), out.data_ptr(), dtype_code(out.dtype), N // 2, _p(colscale),
-                               _p(colbias), M, N, K, TENSOR_CORE_MIN_ROWS, GLU_ACTS[act], _stream())
+                               _p(colbias), M, N, K, TENSOR_CORE_MIN_ROWS, DENSE_ACTS[act], float(limit), float(alpha), _stream())
     if rc == 1:                                   # no fused kernel for these operands
         _launches -= 1
         gu = torch.empty((M, N), dtype=torch.float32, device=a.device)
         linear(a, w, gu, colscale, colbias)
-        glu(gu, out, act, interleaved=True)
+        glu(gu, out, act, interleaved=True, limit=limit, alpha=alpha)
     elif rc != 0:
         raise KernelError(f"tlc_linear_swiglu: {lib.tlc_last_error().decode()}")
 
@@ -646,12 +659,29 @@ def rope_kv_store(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: 
           T, H, KV, hd, int(bool(write_kv)), _stream())
 
 
+def visible_bound(max_keys: int, window: int, chunk: int, keep_first: int, rows: int) -> int:
+    """How many key positions, counted from the page of the first visible one, `rows` consecutive rows of a sequence of at
+    most max_keys positions can see: all of them, or with a window or chunks (and no first keys kept) what those leave."""
+    sizes = [int(s) for s in (window, chunk) if s and int(s) > 0]
+    return int(max_keys) if not sizes or keep_first > 0 else min(int(max_keys), min(sizes) + PAGE - 1 + rows - 1)
+
+
+def _head_gate(gate: Optional[torch.Tensor], T: int, H: int, what: str):
+    """(pointer, row stride) of an optional gate of one number per row and head."""
+    if gate is None:
+        return None, 0
+    if gate.dtype != torch.float32 or tuple(gate.shape) != (T, H):
+        raise KernelError(f"{what}: the heads' gate must be float32 [T, H]")
+    return gate.data_ptr(), _rows(gate, "heads' gate")
+
+
 def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
               positions: torch.Tensor, row_seq: torch.Tensor, slots: torch.Tensor, out: torch.Tensor, H: int, KV: int,
               hd: int, scale: float, window: int = 0, decode_max_keys: int = 0,
               cu_seqlens: Optional[torch.Tensor] = None, start_pos: Optional[torch.Tensor] = None,
               max_keys: int = 0, max_blocks: int = 0, key_ranges: int = 0, softcap: float = 0.0, sink: bool = False,
-              keep_first: int = 0, sink_values: Optional[torch.Tensor] = None) -> None:
+              keep_first: int = 0, sink_values: Optional[torch.Tensor] = None, chunk: int = 0,
+              head_gate: Optional[torch.Tensor] = None) -> None:
     """Causal grouped-query attention of every row over its sequence's pages (keys 0..position,
     or the last `window` of them).  decode_max_keys > 0 says that the rows are single-token
     steps of sequences no longer than that: keys are then split across blocks.  With
@@ -664,25 +694,30 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
     softcap * tanh(score / softcap) after the scale; sink: the softmax's denominator has one more term of score 0, which
     carries no value (both served by the tcgen05 kernel of prompts, the warp kernels and the split-key kernels of single
     tokens).  sink_values float32 [H]: the sink's score per head instead of 0 (implies sink; the score is taken as it is, not
-    scaled).  keep_first > 0 (with a window): the first keep_first keys of a sequence stay visible to every later query."""
-    _gpu(q, k_pages, v_pages, block_table, positions, row_seq, slots, out, sink_values)
+    scaled).  keep_first > 0 (with a window): the first keep_first keys of a sequence stay visible to every later query.
+    chunk > 0: a row sees the keys of its own chunk of that many positions, counted from the sequence's start.  head_gate
+    (float32 [T, H], a range of the columns of a wider projection will do): head h of row t's result is multiplied by the
+    sigmoid of its number."""
+    _gpu(q, k_pages, v_pages, block_table, positions, row_seq, slots, out, sink_values, head_gate)
     T = q.shape[0]
     if sink_values is not None:
         _f32vec(sink_values, H, "attention sink scores")
         sink = True
-    keep_first = int(keep_first) if window else 0
+    keep_first, chunk = int(keep_first) if window else 0, int(chunk or 0)
+    gate = _head_gate(head_gate, T, H, "attention")
     if not q.is_contiguous() or tuple(q.shape) != (T, H * hd) or out.dtype != q.dtype or k_pages.dtype != q.dtype:
         raise KernelError("attention: q must be contiguous [T, H*hd], q and out of the pages' type")
     out_ld = _out_rows(out, T, H * hd, "attention")
     if decode_max_keys > 0 and H // KV <= 8:
-        n_splits = (int(decode_max_keys) + 127) // 128
+        decode_max_keys = visible_bound(decode_max_keys, window, chunk, keep_first, 1)
+        n_splits = (decode_max_keys + 127) // 128
         part_o = torch.empty((T, H, n_splits, hd), dtype=torch.float32, device=q.device)
         part_ml = torch.empty((T, H, n_splits, 2), dtype=torch.float32, device=q.device)
         _call("tlc_attention_decode", q.data_ptr(), dtype_code(q.dtype), k_pages.data_ptr(), v_pages.data_ptr(),
               block_table.data_ptr(), block_table.shape[1], positions.data_ptr(), row_seq.data_ptr(),
               slots.data_ptr(), out.data_ptr(), part_o.data_ptr(), part_ml.data_ptr(), T, H, KV, hd, float(scale),
               int(window or 0), int(decode_max_keys), out_ld, float(softcap), int(bool(sink)), keep_first, _p(sink_values),
-              _stream())
+              chunk, *gate, _stream())
         return
     own_softmax = softcap > 0 or sink
     tiled = decode_max_keys <= 0 and cu_seqlens is not None and start_pos is not None and q.dtype == torch.bfloat16 \
@@ -691,7 +726,8 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
             and library().tlc_attention_prefill_tc_ok(BF16, hd, H, KV):
         B = slots.numel()
         # few row tiles and many keys (a piece of a long prompt): the keys in ranges that run side by side
-        n_split = key_ranges if key_ranges > 0 else library().tlc_attention_prefill_tc_splits(T // 128 + B, H, int(max_keys))
+        n_split = key_ranges if key_ranges > 0 else library().tlc_attention_prefill_tc_splits(
+            T // 128 + B, H, visible_bound(max_keys, window, chunk, keep_first, 128))
         part_o = part_ml = None
         if n_split > 1:
             part_o = torch.empty((T, H, n_split, hd), dtype=torch.float32, device=q.device)
@@ -700,9 +736,9 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
               block_table.data_ptr(), block_table.shape[1], cu_seqlens.data_ptr(), slots.data_ptr(), start_pos.data_ptr(),
               out.data_ptr(), B, T // 128 + B, H, KV, hd, float(scale), int(window or 0), int(max_keys), T,
               out_ld, int(max_blocks), int(n_split), _p(part_o), _p(part_ml), float(softcap), int(bool(sink)), keep_first,
-              _p(sink_values), _stream())
+              _p(sink_values), chunk, *gate, _stream())
         return
-    if tiled and not own_softmax and keep_first == 0:
+    if tiled and not own_softmax and keep_first == 0 and chunk == 0 and head_gate is None:
         B = slots.numel()
         n_tiles = T // 64 + B
         chunk = ctypes.c_int(0)
@@ -720,7 +756,7 @@ def attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, blo
     _call("tlc_attention", q.data_ptr(), dtype_code(q.dtype), k_pages.data_ptr(), v_pages.data_ptr(),
           block_table.data_ptr(), block_table.shape[1], positions.data_ptr(), row_seq.data_ptr(), slots.data_ptr(),
           out.data_ptr(), T, H, KV, hd, float(scale), int(window or 0), out_ld, float(softcap), int(bool(sink)), keep_first,
-          _p(sink_values), _stream())
+          _p(sink_values), chunk, *gate, _stream())
 
 
 DISABLE_FUSED_DECODE_ATTENTION = bool(int(os.environ.get("TLC_DISABLE_FUSED_DECODE_ATTENTION", "0")))
@@ -746,12 +782,14 @@ def attention_decode_fused(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int
                            positions: torch.Tensor, row_seq: torch.Tensor, slots: torch.Tensor, out: torch.Tensor,
                            H: int, KV: int, hd: int, scale: float, window: int, max_keys: int,
                            arrivals: torch.Tensor, softcap: float = 0.0, sink: bool = False, keep_first: int = 0,
-                           sink_values: Optional[torch.Tensor] = None) -> None:
+                           sink_values: Optional[torch.Tensor] = None, chunk: int = 0,
+                           head_gate: Optional[torch.Tensor] = None) -> None:
     """Single-token steps in one kernel: rotates the row's queries and new key (2 * len(inv_freq)
     leading dims of each head), stores the new key/value row into its page when write_kv, attends
     over the sequence's pages and writes out [T, H*hd] bfloat16.  qkv is float32 with dense rows.
-    arrivals: the caller's counters (new_arrival_counters).  softcap, sink, keep_first and sink_values as in attention()."""
-    _gpu(qkv, k_pages, v_pages, inv_freq, block_table, positions, row_seq, slots, out, sink_values)
+    arrivals: the caller's counters (new_arrival_counters).  softcap, sink, keep_first, sink_values, chunk and head_gate as
+    in attention()."""
+    _gpu(qkv, k_pages, v_pages, inv_freq, block_table, positions, row_seq, slots, out, sink_values, head_gate)
     if sink_values is not None:
         _f32vec(sink_values, H, "attention sink scores")
         sink = True
@@ -769,7 +807,9 @@ def attention_decode_fused(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int
     if max(q_off + H * hd, k_off + KV * hd, v_off + KV * hd) > max(ld, qkv.shape[1]):
         raise KernelError("attention_decode_fused: q, k or v lies outside the projection's row")
     _f32vec(inv_freq, inv_freq.numel(), "rope inv_freq")
-    n_splits = (int(max_keys) + 127) // 128
+    keep_first, chunk = int(keep_first) if window else 0, int(chunk or 0)
+    max_keys = visible_bound(max_keys, window, chunk, keep_first, 1)
+    n_splits = (max_keys + 127) // 128
     part_o = torch.empty((T, H, n_splits, hd), dtype=torch.float32, device=qkv.device)
     part_ml = torch.empty((T, H, n_splits, 2), dtype=torch.float32, device=qkv.device)
     _gpu(arrivals)
@@ -781,7 +821,8 @@ def attention_decode_fused(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int
           inv_freq.data_ptr(), 2 * inv_freq.numel(), int(bool(write_kv)), block_table.data_ptr(), block_table.shape[1],
           positions.data_ptr(), row_seq.data_ptr(), slots.data_ptr(), out.data_ptr(), part_o.data_ptr(),
           part_ml.data_ptr(), arrivals.data_ptr(), T, H, KV, hd, float(scale), int(window or 0), int(max_keys), out_ld,
-          float(softcap), int(bool(sink)), int(keep_first) if window else 0, _p(sink_values), _stream())
+          float(softcap), int(bool(sink)), keep_first, _p(sink_values), chunk, *_head_gate(head_gate, T, H, "attention_decode_fused"),
+          _stream())
 
 
 def attention_decode_fused_passes(passes: int) -> None:
@@ -967,13 +1008,14 @@ MAX_LATENT = 512          # latent_attention.cu: 32 * LAT_MAXV values of a laten
 
 def latent_prepare(proj: Optional[torch.Tensor], q_off: int, dkv_off: Optional[int], norm_weight: Optional[torch.Tensor], eps: float,
                    inv_freq: torch.Tensor, step, block_table: torch.Tensor, pages: torch.Tensor, qn: torch.Tensor,
-                   qa: torch.Tensor, H: int, dn: int, r: int, R: int, q_proj: Optional[torch.Tensor] = None) -> None:
+                   qa: torch.Tensor, H: int, dn: int, r: int, R: int, q_proj: Optional[torch.Tensor] = None,
+                   amplitude: float = 1.0) -> None:
     """From a row's projections (float32 [T, *]: H heads of (dn | r) query values at q_off, R + r down-projected values
     at dkv_off, None for a layer that reads another layer's rows; q_proj: the buffer that holds the queries, where it
     is not proj itself, which may then be None with dkv_off None): the unrotated query parts to qn [T, H*dn], the
     rotated ones into the last r columns of every head of qa [T, H*(R+r)], and the cache row [rmsnorm(c) * norm_weight
     | rotated kr] into its page of pages [n, 64, R+r].  The rotation turns interleaved pairs of the first
-    2 * len(inv_freq) dimensions."""
+    2 * len(inv_freq) dimensions; amplitude multiplies every cosine and sine."""
     if q_proj is None:
         q_proj = proj
     if proj is None:
@@ -997,7 +1039,7 @@ def latent_prepare(proj: Optional[torch.Tensor], q_off: int, dkv_off: Optional[i
           -1 if dkv_off is None else int(dkv_off),
           _p(norm_weight), float(eps), inv_freq.data_ptr(), 2 * inv_freq.numel(), step.positions.data_ptr(),
           step.row_seq.data_ptr(), step.slots.data_ptr(), block_table.data_ptr(), block_table.shape[1], pages.data_ptr(),
-          qn.data_ptr(), qa.data_ptr(), dtype_code(pages.dtype), T, H, dn, r, R, _stream())
+          qn.data_ptr(), qa.data_ptr(), dtype_code(pages.dtype), T, H, dn, r, R, float(amplitude), _stream())
 
 
 _latent_tc = not bool(int(os.environ.get("TLC_DISABLE_LATENT_TC", "0")))
@@ -1011,13 +1053,16 @@ def latent_attention_tc(on: bool) -> None:
 
 
 def latent_attention(qa: torch.Tensor, pages: torch.Tensor, sink: Optional[torch.Tensor], block_table: torch.Tensor, step,
-                     out: torch.Tensor, H: int, R: int, r: int, scale: float, key_ranges: int = 0, window: int = 0) -> None:
+                     out: torch.Tensor, H: int, R: int, r: int, scale: float, key_ranges: int = 0, window: int = 0,
+                     head_gate: Optional[torch.Tensor] = None) -> None:
     """out [T, H*R]: every head's softmax-weighted sum of the latents of keys 0..position (with window > 0: of the last
     `window` of them), scores (qa . [c | kr]) * scale, with the head's sink (None: no sink) in the denominator.  bfloat16 rows of sizes the tensor-core kernel is built for take it (all
     heads of a row share every page read); key_ranges > 0 fixes into how many ranges it cuts a tile's keys (0: chosen:
-    more than one for few rows over many keys)."""
-    _gpu(qa, pages, sink, block_table, out)
+    more than one for few rows over many keys).  head_gate (float32 [T, H]): head h of row t's sum is multiplied by the sigmoid
+    of its number (which commutes with whatever linear map is applied to the sum afterwards)."""
+    _gpu(qa, pages, sink, block_table, out, head_gate)
     T = qa.shape[0]
+    gate = _head_gate(head_gate, T, H, "latent_attention")
     _i32(block_table, "block_table")
     _f32vec(sink, H, "attention sink")
     if qa.dtype != pages.dtype or out.dtype != pages.dtype or not qa.is_contiguous() or not out.is_contiguous() \
@@ -1040,11 +1085,11 @@ def latent_attention(qa: torch.Tensor, pages: torch.Tensor, sink: Optional[torch
         _call("tlc_latent_attention_tc", qa.data_ptr(), pages.data_ptr(), _p(sink), block_table.data_ptr(),
               block_table.shape[1], step.cu_seqlens.data_ptr(), step.slots.data_ptr(), step.start_pos.data_ptr(),
               out.data_ptr(), _p(part_o), _p(part_ml), B, T, pairs, n_tiles, H, R, r, float(scale), int(n_split), int(window or 0),
-              _stream())
+              *gate, _stream())
         return
     _call("tlc_latent_attention", qa.data_ptr(), pages.data_ptr(), dtype_code(pages.dtype), _p(sink),
           block_table.data_ptr(), block_table.shape[1], step.positions.data_ptr(), step.row_seq.data_ptr(),
-          step.slots.data_ptr(), out.data_ptr(), T, H, R, r, float(scale), int(window or 0), _stream())
+          step.slots.data_ptr(), out.data_ptr(), T, H, R, r, float(scale), int(window or 0), *gate, _stream())
 
 
 _grouped_mma = not bool(int(os.environ.get("TLC_DISABLE_GROUPED_MMA", "0")))
@@ -1152,6 +1197,23 @@ def moe_route(logits: torch.Tensor, n_experts: int, top: int, tile_rows: int = 3
     return ids, wts, order, offsets, tile_off, int(tile_rows)
 
 
+def moe_route_table(tokens: torch.Tensor, table: torch.Tensor, n_experts: int, weight: float, tile_rows: int = 32):
+    """Routing without a router: row t's experts are table[tokens[t]] (int32 [V, top], the entries of a row distinct and below
+    n_experts), every one of them with the same weight.  Returns what moe_route does."""
+    _gpu(tokens, table)
+    _i32(tokens, "tokens")
+    _i32(table, "expert table")
+    T, (V, top) = tokens.numel(), table.shape
+    ints = torch.empty(2 * T * top + 2 * (n_experts + 1), dtype=torch.int32, device=tokens.device)
+    ids, order = ints[:T * top], ints[T * top:2 * T * top]
+    offsets = ints[2 * T * top:2 * T * top + n_experts + 1]
+    tile_off = ints[2 * T * top + n_experts + 1:]
+    wts = torch.empty(T * top, dtype=torch.float32, device=tokens.device)
+    _call("tlc_moe_route_table", tokens.data_ptr(), table.data_ptr(), T, V, int(n_experts), top, float(weight), ids.data_ptr(),
+          wts.data_ptr(), order.data_ptr(), offsets.data_ptr(), tile_off.data_ptr(), int(tile_rows), _stream())
+    return ids, wts, order, offsets, tile_off, int(tile_rows)
+
+
 def moe_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, routing, top: int, act: torch.Tensor,
                 y: torch.Tensor, act_fn: str = "silu", weight_on: str = "input", limit: float = 0.0, alpha: float = 1.0) -> None:
     """y[t, k, :] for every chosen (token, expert) pair: expert_k(weight * x[t]) with weight_on "input", weight *
@@ -1200,9 +1262,10 @@ def moe_identity(x: torch.Tensor, routing, top: int, n_experts: int, y: torch.Te
 
 
 def qk_whole_norm(qkv: torch.Tensor, q_off: int, q_n: int, q_weight: torch.Tensor, k_off: int, k_n: int, k_weight: torch.Tensor,
-                  eps: float) -> None:
+                  eps: float, q_count: Optional[int] = None, k_count: Optional[int] = None) -> None:
     """In place on the float32 projection: its q_n query columns from q_off (all heads together) become
-    q / sqrt(mean(q^2) + eps) * q_weight, its k_n key columns from k_off likewise."""
+    q / sqrt(mean(q^2) + eps) * q_weight, its k_n key columns from k_off likewise.  q_count, k_count: how many of the columns
+    the mean is over (default all; the others, of padded heads, are zero and have zero weights)."""
     _gpu(qkv, q_weight, k_weight)
     ld = _rows(qkv, "qkv")
     if qkv.dtype != torch.float32 or max(q_off + q_n, k_off + k_n) > max(ld, qkv.shape[1]):
@@ -1210,7 +1273,7 @@ def qk_whole_norm(qkv: torch.Tensor, q_off: int, q_n: int, q_weight: torch.Tenso
     _f32vec(q_weight, q_n, "query norm weight")
     _f32vec(k_weight, k_n, "key norm weight")
     _call("tlc_qk_whole_norm", qkv.data_ptr(), ld, int(q_off), int(q_n), q_weight.data_ptr(), int(k_off), int(k_n),
-          k_weight.data_ptr(), float(eps), qkv.shape[0], _stream())
+          k_weight.data_ptr(), float(eps), qkv.shape[0], int(q_count or q_n), int(k_count or k_n), _stream())
 
 
 # ---- time mixing with a decaying matrix state -------------------------------------------------------------------

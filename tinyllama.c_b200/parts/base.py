@@ -16,7 +16,8 @@ Position      rotation_table() -> inverse frequencies (the kernels rotate q and 
               transform(qkv, q_off, k_off, step, n_heads, n_kv, head_dim): changes the q and k columns of
               the 32-bit projection in place; storing keys and values is the mixer's business
 Mixer         forward(normed [T, D], step, cache, residual [T, D] float32)  adds its output into residual
-FeedForward   forward(normed [T, D], residual [T, D] float32)               adds its output into residual
+FeedForward   forward(normed [T, D], residual [T, D] float32)               adds its output into residual (one that says
+              takes_tokens = True is also given the rows' token ids, tokens=)
 All of them   weight_specs() -> [WeightSpec], bind(tensors, dtype, device)
 Mixers also   cache_requests() -> [KVRequest | StateRequest], step_requests() -> [ChunkRequest]
 """
@@ -32,10 +33,12 @@ import torch
 @dataclass(frozen=True)
 class WeightSpec:
     """One named tensor of a part.  ``init`` tells the random-weights mode how to draw it:
-    normal | ones | zeros | a_log | dt_bias | d_skip."""
+    normal | ones | zeros | a_log | dt_bias | d_skip | near_zero | unit_interval | conv | choices.  below > 0: an integer
+    tensor whose values are 0 .. below - 1, the entries of a row distinct (init "choices")."""
     name: str
     shape: Tuple[int, ...]
     init: str = "normal"
+    below: int = 0
 
 
 # ---- cache needs --------------------------------------------------------------------------
@@ -50,6 +53,8 @@ class KVRequest:
                                 # from the same row (a shared latent) asks for no second set of pages
     keep_first: int = 0         # with a window: the first keep_first positions stay visible to every later query, so the
                                 # pages that hold them are never given back
+    chunk: int = 0              # > 0: a query sees the positions of its own chunk of that many only (counted from the sequence's
+                                # start); pages of chunks that are over are given back
 
 
 @dataclass(frozen=True)
@@ -228,11 +233,13 @@ class LayerRun:
     storing into it.  ``kv_cache`` names an entry whose keys and values (only those) this entry
     reads without storing, while it keeps fixed-size state of its own: a layer that attends over
     what another layer cached.  ``add`` = (table, row) names a learned table of the model ([rows, width]) whose row is added
-    to the residual stream right before this entry runs (a range of layers that repeats marks each pass this way)."""
+    to the residual stream right before this entry runs (a range of layers that repeats marks each pass this way).
+    ``add_embedding``: the embedding output (what the first entry of the run order reads) is added instead."""
     layer: int
     cache: Optional[int] = None
     kv_cache: Optional[int] = None
     add: Optional[Tuple[str, int]] = None
+    add_embedding: bool = False
 
     @property
     def writes(self) -> bool:

@@ -237,7 +237,11 @@ class Block(Part):
         return (self._pre_norm(self.mixer_norm, x32, "block.normed", step, cache),
                 self._pre_norm(self.ffn_norm, x32, "block.ffn_normed", step, cache))
 
-    def _two_branches(self, normed: torch.Tensor, x32: torch.Tensor, run_mixers, ffn_in: Optional[torch.Tensor] = None) -> None:
+    def _ffn_more(self, step: StepInfo) -> dict:
+        """What the feed-forward is given beside its input: the rows' token ids, where it asks for them."""
+        return {"tokens": step.tokens} if getattr(self.ffn, "takes_tokens", False) else {}
+
+    def _two_branches(self, normed: torch.Tensor, x32: torch.Tensor, run_mixers, ffn_in: Optional[torch.Tensor], more: dict) -> None:
         """A parallel layer on two streams (under stream capture: two branches of the graph): the mixers, which add
         their outputs into the residual stream, and the feed-forward's terms; the terms are added after the branches have
         met, on the current stream, so the order of the sums is fixed.  run_mixers(): launches the mixers on whatever
@@ -256,12 +260,12 @@ class Block(Part):
             if PARALLEL_FFN == 1:
                 run_mixers()
             else:
-                terms = self.ffn.forward_parts(normed if ffn_in is None else ffn_in)
+                terms = self.ffn.forward_parts(normed if ffn_in is None else ffn_in, **more)
             self._ffn_done.record(side)
         finally:
             torch.cuda.set_stream(main)
         if PARALLEL_FFN == 1:
-            terms = self.ffn.forward_parts(normed if ffn_in is None else ffn_in)
+            terms = self.ffn.forward_parts(normed if ffn_in is None else ffn_in, **more)
         else:
             run_mixers()
         main.wait_event(self._ffn_done)
@@ -354,12 +358,12 @@ class Block(Part):
             normed, ffn_in = self._parallel_inputs(x32, step, cache) if self.parallel_ffn \
                 else (self._pre_norm(self.mixer_norm, x32, "block.normed", step, cache), None)
             if self._beside(x32, step):
-                self._two_branches(normed, x32, lambda: self._run_mixers(normed, x32, step, cache), ffn_in)
+                self._two_branches(normed, x32, lambda: self._run_mixers(normed, x32, step, cache), ffn_in, self._ffn_more(step))
                 return False
             self._run_mixers(normed, x32, step, cache)
         if self.parallel_ffn:
             # h was normed before the mixers added anything; the sum x + mixers(h) + ffn(h) forms in the residual stream
-            self.ffn.forward(ffn_in, x32)
+            self.ffn.forward(ffn_in, x32, **self._ffn_more(step))
             return False
         if self.ffn is not None:
             return self._feed_forward(x32, step, cache, copy_for_next)
@@ -392,7 +396,9 @@ class Block(Part):
         copy = self._stream_copy("block.normed", x32) if copy_for_next and self.ffn_out_norm is not None else None
         self._copied.discard("block.normed")          # (the next layer is told by the return value)
         # without a norm in front, a feed-forward that can use them (takes_stream) also gets the 32-bit rows themselves
-        more = {"stream": x32} if getattr(self.ffn_norm, "identity", False) and getattr(self.ffn, "takes_stream", False) else {}
+        more = self._ffn_more(step)
+        if getattr(self.ffn_norm, "identity", False) and getattr(self.ffn, "takes_stream", False):
+            more["stream"] = x32
         if self.ffn_out_norm is None:
             self.ffn.forward(normed, x32, **more)
         elif hasattr(self.ffn, "forward_parts"):
@@ -402,9 +408,9 @@ class Block(Part):
         else:
             y = scratch_buf("block.ffn_out", x32.shape, torch.float32, x32.device)
             if self._ffn_overwrites:
-                self.ffn.forward(normed, y, accumulate=False)
+                self.ffn.forward(normed, y, accumulate=False, **more)
             else:
                 y.zero_()
-                self.ffn.forward(normed, y)
+                self.ffn.forward(normed, y, **more)
             self.ffn_out_norm.add_normed(y, x32, copy=copy)
         return copy is not None

@@ -23,7 +23,7 @@ class SwiGLU(Part):
                  down_scale: float = 1.0, act: str = "silu", names: Optional[Dict[str, str]] = None, limit: float = 0.0,
                  alpha: float = 1.0):
         """act: "silu", "gelu_tanh", or "swish_clamped": with g = min(W_gate h, limit) and u = W_up h held within +-limit,
-        g * sigmoid(alpha g) * (u + 1) (the product and the activation are then two kernels).  names: tensor names of gate, up, down after the prefix (default: the
+        g * sigmoid(alpha g) * (u + 1).  names: tensor names of gate, up, down after the prefix (default: the
         gate_proj.weight / up_proj.weight / down_proj.weight of the architecture's checkpoints; biases, where asked
         for, are those names with .bias for .weight)."""
         self.hidden, self.F = int(hidden), int(intermediate)
@@ -51,7 +51,7 @@ class SwiGLU(Part):
         self.down.bind(tensors, dtype, device)
         # Rows regrouped as 8 gate rows followed by their 8 up rows, so that the product's epilogue
         # has a feature's gate and up side by side and writes silu(gate) * up directly.
-        self.interleaved = self.F % 8 == 0 and self.act in ops.GLU_ACTS
+        self.interleaved = self.F % 8 == 0
         if self.interleaved:
             F = self.F
             idx = torch.arange(2 * F, device=self.gate_up.weight.device).reshape(2, F // 8, 8).permute(1, 0, 2).reshape(-1)
@@ -66,7 +66,8 @@ class SwiGLU(Part):
         T = normed.shape[0]
         act = scratch_buf("swiglu.act", (T, self.F), normed.dtype, normed.device)
         if self.interleaved:
-            ops.linear_swiglu(normed, self.gate_up.weight, act, self.gate_up.colscale, self.gate_up.colbias, self.act)
+            ops.linear_swiglu(normed, self.gate_up.weight, act, self.gate_up.colscale, self.gate_up.colbias, self.act,
+                              self.limit, self.alpha)
         else:
             gu = scratch_buf("swiglu.gate_up", (T, 2 * self.F), torch.float32, normed.device)
             self.gate_up.forward(normed, gu)
@@ -154,14 +155,25 @@ class MoEFeedForward(Part):
     expert is chosen by its score plus a learned correction (choice_bias_name) and weighted by the score alone, not
     renormalised.  n_identity > 0: the router has that many more outputs than there are experts; the last n_identity stand for
     experts that return their input (times the weight) and have no tensors.  act="relu_squared": experts without a gate,
-    W_down max(W_up h, 0)^2 (expert_names gives up and down only; the weight goes on the output)."""
+    W_down max(W_up h, 0)^2 (expert_names gives up and down only; the weight goes on the output).  table_name instead of a
+    router: an integer tensor [vocab, top] gives every token id its experts, each weighted 1 / top; nothing is scored.  A shared
+    expert without a gate (shared_gate_name None) is added as it is."""
 
-    def __init__(self, hidden: int, n_experts: int, top: int, expert_ff: int, router_name: str, expert_names: Dict[str, str],
+    def __init__(self, hidden: int, n_experts: int, top: int, expert_ff: int, router_name: Optional[str], expert_names: Dict[str, str],
                  shared: Optional[PartSpec] = None, shared_gate_name: Optional[str] = None, router_bias_name: Optional[str] = None,
                  weights: str = "sigmoid", weight_on: str = "input", act: str = "silu", limit: float = 0.0, alpha: float = 1.0,
-                 choice_bias_name: Optional[str] = None, n_identity: int = 0, weights_sum_to: float = 0.0):
+                 choice_bias_name: Optional[str] = None, n_identity: int = 0, weights_sum_to: float = 0.0,
+                 table_name: Optional[str] = None, vocab: int = 0):
         """expert_names: patterns of gate, up, down with {e} for the expert's index.  weights_sum_to > 0 (weights
-        "softmax_all"): a token's weights are the chosen scores divided by their sum (+ 1e-20) times this number."""
+        "softmax_all"): a token's weights are the chosen scores divided by their sum (+ 1e-20) times this number.
+        table_name: the tensor [vocab, top] that routes by token id (router_name is then None)."""
+        self.table_name, self.vocab, self.takes_tokens = table_name, int(vocab), table_name is not None
+        if (table_name is None) == (router_name is None):
+            raise ValueError("moe: a router or a table chooses the experts")
+        if table_name is not None and (self.vocab < 1 or router_bias_name or choice_bias_name or n_identity or shared_gate_name
+                                       or weights_sum_to):
+            raise ValueError("moe: a table of experts needs the vocabulary's size and takes no router's biases, identity outputs, "
+                             "weights to be normed or gated shared expert")
         self.weights_sum_to = float(weights_sum_to)
         if self.weights_sum_to < 0 or (self.weights_sum_to and weights != "softmax_all"):
             raise ValueError("moe: weights normed to a sum go with weights 'softmax_all' and a positive sum")
@@ -184,12 +196,13 @@ class MoEFeedForward(Part):
             raise ValueError(f"moe: {self.top} of {self.n_out} router outputs cannot be chosen")
         self.router_name, self.expert_names, self.shared_gate_name = router_name, dict(expert_names), shared_gate_name
         self.shared = shared.build() if shared is not None else None
-        if (self.shared is None) != (shared_gate_name is None):
-            raise ValueError("moe: a shared expert and its gate come together")
+        if self.shared is None and shared_gate_name is not None:
+            raise ValueError("moe: a shared expert's gate needs a shared expert")
         self.dtype = None
 
     def weight_specs(self) -> List[WeightSpec]:
-        specs = [WeightSpec(self.router_name, (self.n_out, self.hidden))]
+        specs = [WeightSpec(self.router_name, (self.n_out, self.hidden))] if self.router_name else \
+            [WeightSpec(self.table_name, (self.vocab, self.top), "choices", below=self.E)]
         if self.router_bias_name:
             specs.append(WeightSpec(self.router_bias_name, (self.n_out,)))
         if self.choice_bias_name:
@@ -200,7 +213,9 @@ class MoEFeedForward(Part):
                 specs.append(WeightSpec(n["gate"], (self.F, self.hidden)))
             specs += [WeightSpec(n["up"], (self.F, self.hidden)), WeightSpec(n["down"], (self.hidden, self.F))]
         if self.shared is not None:
-            specs += self.shared.weight_specs() + [WeightSpec(self.shared_gate_name, (1, self.hidden))]
+            specs += self.shared.weight_specs()
+            if self.shared_gate_name:
+                specs.append(WeightSpec(self.shared_gate_name, (1, self.hidden)))
         return specs
 
     def bind(self, tensors: Dict[str, torch.Tensor], dtype, device) -> None:
@@ -209,9 +224,15 @@ class MoEFeedForward(Part):
         # The router's logits are 32-bit sums.  A weight stored in bfloat16 times an input rounded to bfloat16 has an exact
         # 32-bit product, so the bfloat16 product with 32-bit accumulation IS the 32-bit result and a bfloat16 run keeps
         # such a router in bfloat16 (the tensor cores); a router stored in 32-bit, and every 32-bit run, multiplies in 32-bit.
-        rows = [tensors[self.router_name]] + ([tensors[self.shared_gate_name]] if self.shared is not None else [])
+        rows = [tensors[n] for n in (self.router_name, self.shared_gate_name) if n]
         rdt = torch.bfloat16 if all(matrix_dtype(r.dtype, dtype) == torch.bfloat16 for r in rows) else torch.float32
-        self.router = torch.cat([r.to(device=device, dtype=rdt) for r in rows], dim=0).contiguous()
+        self.router = torch.cat([r.to(device=device, dtype=rdt) for r in rows], dim=0).contiguous() if rows else None
+        self.table = None
+        if self.table_name:
+            table = tensors[self.table_name]
+            if table.numel() and (int(table.min()) < 0 or int(table.max()) >= self.E):
+                raise ValueError(f"moe: '{self.table_name}' names experts outside 0..{self.E - 1}")
+            self.table = table.to(device=device, dtype=torch.int32).contiguous()
         self.router_bias = None
         if self.router_bias_name:                # added to the 32-bit logits in the product's epilogue (nothing on the shared gate's)
             self.router_bias = torch.zeros(self.router.shape[0], dtype=torch.float32, device=device)
@@ -235,16 +256,24 @@ class MoEFeedForward(Part):
 
     takes_stream = True        # forward(..., stream=x32): an expert that returns its input returns the 32-bit rows
 
-    def forward_parts(self, normed: torch.Tensor, stream: Optional[torch.Tensor] = None):
+    def _route(self, normed: torch.Tensor, tokens: Optional[torch.Tensor]):
+        """(routing as moe_experts takes it, the router's logits or None)."""
+        tile_rows = ops.moe_tile_rows(normed, self.w_gate_up, self.dtype, self.top, self.F)
+        if self.table is not None:
+            if tokens is None:
+                raise ValueError("moe: experts chosen by a table need the rows' token ids")
+            return ops.moe_route_table(tokens, self.table, self.E, 1.0 / self.top, tile_rows), None
+        logits = scratch_buf("moe.logits", (normed.shape[0], self.router.shape[0]), torch.float32, normed.device)
+        ops.linear(normed, self.router, logits, None, self.router_bias)
+        return ops.moe_route(logits, self.n_out, self.top, tile_rows, self.weights, self.choice_bias, self.n_identity,
+                             self.weights_sum_to), logits
+
+    def forward_parts(self, normed: torch.Tensor, stream: Optional[torch.Tensor] = None, tokens: Optional[torch.Tensor] = None):
         """(parts float32 [T, top, D], shared expert's output float32 [T, D] or None, its gate's logit float32 [T] or
-        None): the result is sum_k parts[:, k] + sigmoid(logit) * shared.  stream: the 32-bit rows that `normed` is a
+        None): the result is sum_k parts[:, k] + sigmoid(logit) * shared (without a gate: + shared).  stream: the 32-bit rows that `normed` is a
         copy of, where the layer has no norm in front of this part (identity experts then return those)."""
         T, dev = normed.shape[0], normed.device
-        n_logits = self.router.shape[0]
-        logits = scratch_buf("moe.logits", (T, n_logits), torch.float32, dev)
-        ops.linear(normed, self.router, logits, None, self.router_bias)
-        routing = ops.moe_route(logits, self.n_out, self.top, ops.moe_tile_rows(normed, self.w_gate_up, self.dtype, self.top, self.F),
-                                self.weights, self.choice_bias, self.n_identity, self.weights_sum_to)
+        routing, logits = self._route(normed, tokens)
         act = scratch_buf("moe.act", (T * self.top, self.F), self.dtype, dev)
         parts = scratch_buf("moe.parts", (T, self.top, self.hidden), torch.float32, dev)
         ops.moe_experts(normed, self.w_gate_up, self.w_down, routing, self.top, act, parts, self.act, self.weight_on, self.limit,
@@ -255,7 +284,8 @@ class MoEFeedForward(Part):
             return parts, None, None
         shared_out = scratch_buf("moe.shared", (T, self.hidden), torch.float32, dev)
         self.shared.forward(normed, shared_out, accumulate=False)
-        return parts, shared_out, logits[:, self.n_out]      # the gate's logit: whoever adds the terms takes its sigmoid
+        # the gate's logit: whoever adds the terms takes its sigmoid
+        return parts, shared_out, logits[:, self.n_out] if self.shared_gate_name else None
 
     def add_parts(self, terms, residual: torch.Tensor, accumulate: bool = True) -> None:
         """Adds what forward_parts returned into `residual` (a token's terms in the order of its choices).  A block that
@@ -264,5 +294,5 @@ class MoEFeedForward(Part):
         ops.rmsnorm_add(parts, None, 0.0, residual, extra, gate, gate_sigmoid=True, accumulate=accumulate)
 
     def forward(self, normed: torch.Tensor, residual: torch.Tensor, accumulate: bool = True,
-                stream: Optional[torch.Tensor] = None) -> None:
-        self.add_parts(self.forward_parts(normed, stream), residual, accumulate)
+                stream: Optional[torch.Tensor] = None, tokens: Optional[torch.Tensor] = None) -> None:
+        self.add_parts(self.forward_parts(normed, stream, tokens), residual, accumulate)

@@ -23,6 +23,8 @@ twice the heads, the queries regrouped so that a map's heads share the map's key
 And: a short causal convolution over time on every channel of the projected q, k and v, before any norm or rotation (the
 last taps - 1 projected rows of a sequence are kept between steps); and values blended with those of another layer, the
 first of the layers that share them, of the same token: v <- (1 - lam) v + lam v_first.
+And: keys of the query's own chunk of so many positions only; an output gate of one number per head (the attention kernels
+multiply by it as they write a head's result); a norm over the whole projection of padded heads.
 """
 from __future__ import annotations
 
@@ -32,7 +34,7 @@ from typing import Dict, List, Optional
 import torch
 
 from ... import ops
-from ..base import KVRequest, LayerCache, Part, PartSpec, StateRequest, StepInfo, WeightSpec, act_empty, register_mixer, scratch_buf, to_vec
+from ..base import KVRequest, LayerCache, Part, PartSpec, StateRequest, StepInfo, WeightSpec, register_mixer, scratch_buf, to_vec
 from ..linear import StackedLinear
 
 
@@ -46,7 +48,7 @@ class AttentionMixer(Part):
                  whole_norm: Optional[Dict[str, object]] = None, softcap: float = 0.0, sink: bool = False,
                  head_norm: Optional[Dict[str, object]] = None, sink_name: Optional[str] = None, keep_first: int = 0,
                  maps: int = 1, difference: Optional[Dict[str, object]] = None, conv_taps: int = 0,
-                 v_mix: Optional[Dict[str, object]] = None):
+                 v_mix: Optional[Dict[str, object]] = None, chunk: Optional[int] = None, gate_per: str = "value"):
         """names: tensor names of q, k, v, o (and g, the gate's projection) after the prefix, where they are not the
         q_proj.weight ... of the architecture's checkpoints (biases then take no part).  scale: what scores are
         multiplied by (default head_dim ** -0.5).  v_dim: size of a value head (default head_dim).  qk_norm_eps: queries
@@ -66,7 +68,9 @@ class AttentionMixer(Part):
         taps], newest tap last) smooth the projected q, k and v along the sequence, y_t = sum_j w[:, j] u_(t - taps + 1 + j),
         before anything else.  v_mix (with conv_taps) = dict(group=any name, first=True) for the layer whose (convolved) values
         the later ones of the group take a share of, dict(group=..., name=tensor of one number lam) for those:
-        v <- (1 - lam) v + lam v_first; the blended v is what is cached."""
+        v <- (1 - lam) v + lam v_first; the blended v is what is cached.  chunk: a query sees the keys of its own chunk of that
+        many positions (counted from the sequence's start).  gate_per "head": the tensor g has a row per head, and head h's
+        result is multiplied by the sigmoid of its number."""
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} heads are not a multiple of {n_kv_heads} key/value heads")
         if not (1 <= int(head_dim) <= ops.MAX_HEAD_DIM):
@@ -90,7 +94,12 @@ class AttentionMixer(Part):
         self.qk_norm_eps = float(qk_norm_eps) if qk_norm_eps is not None else None
         if gate is not None and gate not in ops.GATES:
             raise ValueError(f"attention: unknown output gate '{gate}'; known: {sorted(ops.GATES)}")
-        self.gate = gate
+        if gate_per not in ("value", "head") or (gate_per == "head" and (gate != "sigmoid" or int(maps) != 1)):
+            raise ValueError("attention: a gate is per value, or (a sigmoid, with one map) per head")
+        self.gate, self.gate_per = gate, gate_per
+        self.chunk = int(chunk) if chunk else 0
+        if self.chunk < 0 or (self.chunk and window):
+            raise ValueError("attention: chunks and a window do not go together")
         self.position = position.build()
         layout = getattr(self.position, "layout", "split_half")
         if layout not in ("split_half", "interleaved"):
@@ -122,8 +131,8 @@ class AttentionMixer(Part):
         if self.softcap < 0:
             raise ValueError(f"attention: a score cap of {softcap}")
         self.whole_norm = dict(whole_norm) if whole_norm else None
-        if self.whole_norm and (self.qk_dim != self.hd or not {"q", "k", "eps"} <= set(self.whole_norm)):
-            raise ValueError("attention: a norm over the whole projection needs q, k (weight names) and eps, and unpadded heads")
+        if self.whole_norm and not {"q", "k", "eps"} <= set(self.whole_norm):
+            raise ValueError("attention: a norm over the whole projection needs q, k (weight names) and eps")
         nm = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", o="o_proj.weight")
         nm.update(names or {})
         if self.gate and "g" not in nm:
@@ -145,7 +154,12 @@ class AttentionMixer(Part):
             self.v_off = self.qkv.add(prefix + nm["k"], self.KV * self.hd, b("k_proj"), in_scale)
         else:
             self.v_off = self.qkv.add(prefix + nm["v"], self.KV * self.hd, b("v_proj"), in_scale, heads=v_heads(self.KV), gather=v_rows)
-        self.g_off = self.qkv.add(prefix + nm["g"], self.H * self.hd, None, in_scale, heads=v_heads(self.H)) if self.gate else None
+        self.g_off = None
+        if self.gate and self.gate_per == "value":
+            self.g_off = self.qkv.add(prefix + nm["g"], self.H * self.hd, None, in_scale, heads=v_heads(self.H))
+        elif self.gate:                # a row per head, filled up so that the rows of the projection stay on 16-byte boundaries
+            rows = (self.H + 7) // 8 * 8
+            self.g_off = self.qkv.add(prefix + nm["g"], rows, None, in_scale, heads=(1, self.H, rows))
         self.o = StackedLinear(self.Hq * self.hd, in_heads=v_heads(self.Hq))
         self.o.add(prefix + nm["o"], hidden, b("o_proj"), 1.0, out_scale)
         self.dtype = None
@@ -174,7 +188,7 @@ class AttentionMixer(Part):
         fused = self.dtype == torch.bfloat16 and self.position.rotation_table() is not None \
             and ops.library().tlc_attention_decode_fused_ok(self.H, self.KV, self.hd) \
             and not ops.DISABLE_FUSED_DECODE_ATTENTION
-        return (1 if fused else 3) + int(self.pre_transform) + int(self.gate is not None) + int(self.whole_norm is not None) \
+        return (1 if fused else 3) + int(self.pre_transform) + int(self.gate is not None and self.gate_per == "value") + int(self.whole_norm is not None) \
             + int(self.maps > 1)
 
     @property
@@ -190,8 +204,8 @@ class AttentionMixer(Part):
                 seen.add(sp.name)
                 specs.append(sp)
         if self.whole_norm:
-            specs += [WeightSpec(self.prefix + self.whole_norm["q"], (self.H * self.hd,), "ones"),
-                      WeightSpec(self.prefix + self.whole_norm["k"], (self.KV * self.hd,), "ones")]
+            specs += [WeightSpec(self.prefix + self.whole_norm["q"], (self.H * self.qk_dim,), "ones"),
+                      WeightSpec(self.prefix + self.whole_norm["k"], (self.KV * self.qk_dim,), "ones")]
         if self.head_norm:
             specs += [WeightSpec(self.prefix + self.head_norm["q"], (self.qk_dim,), "ones"),
                       WeightSpec(self.prefix + self.head_norm["k"], (self.qk_dim,), "ones")]
@@ -205,7 +219,8 @@ class AttentionMixer(Part):
         return specs
 
     def cache_requests(self) -> list:
-        reqs = [KVRequest(self.cache_key, self.KV, self.hd, self.window, keep_first=self.keep_first if self.window else 0)]
+        reqs = [KVRequest(self.cache_key, self.KV, self.hd, self.window, keep_first=self.keep_first if self.window else 0,
+                          chunk=self.chunk)]
         if self.conv_taps > 1:
             reqs.append(StateRequest(self.cache_key + ".conv", (self.conv_taps - 1, self.conv_channels)))
         return reqs
@@ -216,8 +231,8 @@ class AttentionMixer(Part):
         self.o.bind(tensors, dtype, device)
         self.position.bind(tensors, dtype, device)
         if self.whole_norm:
-            self.q_norm_w = to_vec(tensors[self.prefix + self.whole_norm["q"]], device)
-            self.k_norm_w = to_vec(tensors[self.prefix + self.whole_norm["k"]], device)
+            self.q_norm_w = self._padded(to_vec(tensors[self.prefix + self.whole_norm["q"]], device), self.H)
+            self.k_norm_w = self._padded(to_vec(tensors[self.prefix + self.whole_norm["k"]], device), self.KV)
         self.q_head_w = self.k_head_w = None
         if self.head_norm:
             self.q_head_w = to_vec(tensors[self.prefix + self.head_norm["q"]], device)
@@ -243,15 +258,22 @@ class AttentionMixer(Part):
         # mixer, model or stream ever shares them; made here, outside any stream capture
         self._arrivals = ops.new_arrival_counters(device) if torch.device(device).type == "cuda" else None
 
+    def _padded(self, w: torch.Tensor, heads: int) -> torch.Tensor:
+        """A weight of heads * qk_dim values laid out over the padded heads, with zeros between."""
+        full = torch.zeros((heads, self.hd), dtype=torch.float32, device=w.device)
+        full[:, :self.qk_dim] = w.reshape(heads, self.qk_dim)
+        return full.reshape(-1).contiguous()
+
     def input_projection(self) -> StackedLinear:
         """What this mixer computes from the normed input before anything else (a block may stack
         the input projections of its mixers into one product)."""
         return self.qkv
 
-    def forward(self, normed: torch.Tensor, step: StepInfo, cache: LayerCache, residual: torch.Tensor) -> None:
-        qkv = act_empty((step.n_rows, self.qkv.out_features), normed, torch.float32)
+    def forward(self, normed: torch.Tensor, step: StepInfo, cache: LayerCache, residual: torch.Tensor, accumulate: bool = True) -> None:
+        """Adds the result into `residual` (float32 [T, D]), or overwrites it with accumulate False."""
+        qkv = scratch_buf(f"attention.{self.cache_key}.qkv", (step.n_rows, self.qkv.out_features), torch.float32, normed.device)
         self.qkv.forward(normed, qkv)
-        self.forward_projected(qkv, step, cache, residual)
+        self.o.forward(self.mix(qkv, step, cache), residual, accumulate=accumulate)
 
     def forward_projected(self, qkv: torch.Tensor, step: StepInfo, cache: LayerCache, residual: torch.Tensor) -> None:
         """qkv: this mixer's input projection, float32 [T, q|k|v] (rows may be strided)."""
@@ -276,7 +298,7 @@ class AttentionMixer(Part):
             qkv = self._convolved(qkv, step, cache)
         if self.whole_norm:           # over all heads at once, before any rotation (the value columns keep the projection)
             ops.qk_whole_norm(qkv, self.q_off, self.H * self.hd, self.q_norm_w, self.k_off, self.KV * self.hd, self.k_norm_w,
-                              float(self.whole_norm["eps"]))
+                              float(self.whole_norm["eps"]), self.H * self.qk_dim, self.KV * self.qk_dim)
         table = self.position.rotation_table()
         if table is None:
             # not a rotation: the part changes q and k in place; what is stored below is its result
@@ -288,6 +310,7 @@ class AttentionMixer(Part):
                                self.q_head_w, self.k_head_w, float(self.head_norm["eps"]) if self.head_norm else 0.0,
                                float(getattr(self.position, "amplitude", 1.0)))
             table = self._no_rotation
+        head_gate = projected[:, self.g_off:self.g_off + self.H] if self.gate and self.gate_per == "head" else None
         joined = out
         if self.maps > 1:             # the kernels write the maps' results; the join writes the heads'
             out = None
@@ -297,7 +320,8 @@ class AttentionMixer(Part):
             ops.attention_decode_fused(qkv, self.q_off, self.k_off, self.v_off, kv.k_pages, kv.v_pages, table,
                                        cache.writes, kv.block_table, step.positions, step.row_seq, step.slots, att,
                                        self.H, self.KV, self.hd, self.scale, self.window or 0,
-                                       step.max_context, self._arrivals, self.softcap, self.sink, self.keep_first, self.sink_values)
+                                       step.max_context, self._arrivals, self.softcap, self.sink, self.keep_first, self.sink_values,
+                                       self.chunk, head_gate)
             return self._joined(self._gated(att, projected), joined)
         q = scratch_buf(f"attention.{self.cache_key}.q", (T, self.H * self.hd), self.dtype, qkv.device)
         ops.rope_kv_store(qkv, self.q_off, self.k_off, self.v_off, q, kv.k_pages, kv.v_pages, table, step.positions,
@@ -306,7 +330,8 @@ class AttentionMixer(Part):
         ops.attention(q, kv.k_pages, kv.v_pages, kv.block_table, step.positions, step.row_seq, step.slots, att,
                       self.H, self.KV, self.hd, self.scale, self.window or 0,
                       step.max_context if step.max_new == 1 else 0, step.cu_seqlens, step.start_pos, step.max_context,
-                      max_blocks, softcap=self.softcap, sink=self.sink, keep_first=self.keep_first, sink_values=self.sink_values)
+                      max_blocks, softcap=self.softcap, sink=self.sink, keep_first=self.keep_first, sink_values=self.sink_values,
+                      chunk=self.chunk, head_gate=head_gate)
         return self._joined(self._gated(att, projected), joined)
 
     def _convolved(self, qkv: torch.Tensor, step: StepInfo, cache: LayerCache) -> torch.Tensor:
@@ -344,7 +369,7 @@ class AttentionMixer(Part):
         return out
 
     def _gated(self, att: torch.Tensor, qkv: torch.Tensor) -> torch.Tensor:
-        if self.gate:
+        if self.gate and self.gate_per == "value":
             ops.gate_mul(att, qkv[:, self.g_off:self.g_off + self.H * self.hd], self.gate)
         return att
 

@@ -15,7 +15,10 @@ down-projection.
 
 Options: no rotated part at all (rot_dim 0 with the position part "none": attention without positions); no sink
 (names without 'sink'); queries through a latent of their own (q_rank: c_q = RMSnorm(W_dq h) * w, q = W_uq c_q, names
-dq, dq_norm, uq instead of q); a sliding window (a row sees itself and the window - 1 rows before it).
+dq, dq_norm, uq instead of q); a sliding window (a row sees itself and the window - 1 rows before it); a rotation whose
+cosines and sines have another amplitude (the position part's business); an output gate of one number per head (names with
+'g'): head i's result times sigmoid((W_g h)_i).  The gate is a number, so it commutes with V_i: the attention kernels multiply
+sum_j p_j c_j by it as they write it.
 """
 from __future__ import annotations
 
@@ -33,7 +36,7 @@ class LatentAttentionMixer(Part):
     def __init__(self, hidden: int, n_heads: int, head_dim: int, rot_dim: int, v_dim: int, kv_rank: int, scale: float,
                  eps: float, position: PartSpec, names: Dict[str, str], own_latent: bool = True, cache_key: str = "latent",
                  q_rank: Optional[int] = None, window: Optional[int] = None, cache_window: Optional[int] = None):
-        """names: tensor names of q (or, with q_rank, of dq, dq_norm, uq), dkv, dkv_norm, uk, uv, o and optionally sink.
+        """names: tensor names of q (or, with q_rank, of dq, dq_norm, uq), dkv, dkv_norm, uk, uv, o and optionally sink and g.
         own_latent False: the layer has no down-projection and reads the rows of the entry that its run-order entry names.
         window: how many keys a row sees, itself included (None: all).  cache_window: how many rows back the cache must
         keep (None: all); a layer whose rows other layers read with windows of their own is given the widest."""
@@ -65,6 +68,10 @@ class LatentAttentionMixer(Part):
             self.q_off = self.proj.add(names["q"], self.H * (self.dn + self.r))
             self.uq = None
         self.dkv_off = self.proj.add(names["dkv"], self.R + self.r) if self.own_latent else None
+        self.g_off = None
+        if self.names.get("g"):       # a row per head, filled up so that the projection's rows stay on 16-byte boundaries
+            rows = (self.H + 7) // 8 * 8
+            self.g_off = self.proj.add(self.names["g"], rows, heads=(1, self.H, rows))
         self.o = StackedLinear(self.H * self.dv)
         self.o.add(names["o"], hidden)
         self.dtype = None
@@ -122,10 +129,11 @@ class LatentAttentionMixer(Part):
             q_proj, q_off = new("q", (T, self.uq.out_features), torch.float32), 0
             self.uq.forward(cq, q_proj)
         ops.latent_prepare(proj, q_off, self.dkv_off, self.c_norm, self.eps, self.position.rotation_table(), step,
-                           kv.block_table, pages, qn, qa, H, dn, r, R, q_proj)
+                           kv.block_table, pages, qn, qa, H, dn, r, R, q_proj, float(getattr(self.position, "amplitude", 1.0)))
         ops.linear_heads(qn, dn, self.uk_t, qa, R + r)                       # qa[:, i, :R] = U_i^T qn_i
         lat = new("lat", (T, H * R), self.dtype)
-        ops.latent_attention(qa, pages, self.sink, kv.block_table, step, lat, H, R, r, self.scale, window=self.window or 0)
+        ops.latent_attention(qa, pages, self.sink, kv.block_table, step, lat, H, R, r, self.scale, window=self.window or 0,
+                             head_gate=None if self.g_off is None else proj[:, self.g_off:self.g_off + H])
         att = new("att", (T, H * dv), self.dtype)
         ops.linear_heads(lat, R, self.uv, att, dv)                           # att[:, i] = V_i (sum_j p_j c_j)
         self.o.forward(att, residual, accumulate=accumulate)

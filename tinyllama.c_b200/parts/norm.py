@@ -16,9 +16,11 @@ from .base import LayerCache, Part, StateRequest, StepInfo, WeightSpec, register
 
 @register_norm("rmsnorm")
 class RMSNorm(Part):
-    def __init__(self, width: int, eps: float, weight_name: str, offset: float = 0.0, one_gain: bool = False):
+    def __init__(self, width: int, eps: float, weight_name: str, offset: float = 0.0, one_gain: bool = False, scale: float = 1.0):
         """offset: what is added to the stored weight (1.0 for a weight stored as its distance from one).  one_gain: the stored
-        weight is a single number for all coordinates (a tensor without dimensions)."""
+        weight is a single number for all coordinates (a tensor without dimensions).  scale: a constant that the normed row is
+        multiplied by (a multiplier on what a sublayer adds to the stream; it folds into the weight)."""
+        self.scale = float(scale)
         self.width, self.eps, self.weight_name, self.offset = int(width), float(eps), weight_name, float(offset)
         self.one_gain = bool(one_gain)
         self.weight: Optional[torch.Tensor] = None
@@ -32,6 +34,8 @@ class RMSNorm(Part):
             self.weight = self.weight.reshape(1).expand(self.width).contiguous()
         if self.offset != 0.0:
             self.weight = (self.weight + self.offset).contiguous()        # in 32 bits
+        if self.scale != 1.0:
+            self.weight = (self.weight * self.scale).contiguous()
 
     def forward(self, x32: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         ops.rmsnorm(x32, self.weight, self.eps, out, rows)

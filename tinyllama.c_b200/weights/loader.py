@@ -51,7 +51,9 @@ def check_tensors(model: Model, tensors: Dict[str, torch.Tensor]) -> None:
         if n in tensors and tuple(tensors[n].shape) != tuple(s.shape):
             wrong.append(f"{n}: expected {list(s.shape)}, found {list(tensors[n].shape)}")
     bad_type = sorted(f"{n}: {tensors[n].dtype}" for n in specs
-                      if n in tensors and not tensors[n].dtype.is_floating_point)
+                      if n in tensors and not tensors[n].dtype.is_floating_point and not specs[n].below)
+    bad_type += sorted(f"{n}: {tensors[n].dtype} (integers expected)" for n in specs
+                       if n in tensors and specs[n].below and tensors[n].dtype.is_floating_point)
     if missing or unexpected or wrong or bad_type:
         lines = [f"weights do not match architecture {model.config.architecture}:"]
         if missing:
@@ -61,7 +63,7 @@ def check_tensors(model: Model, tensors: Dict[str, torch.Tensor]) -> None:
         if wrong:
             lines.append(f"  wrong shapes ({len(wrong)}): " + "; ".join(wrong))
         if bad_type:
-            lines.append(f"  not floating point ({len(bad_type)}): " + "; ".join(bad_type))
+            lines.append(f"  wrong element types ({len(bad_type)}): " + "; ".join(bad_type))
         raise WeightError("\n".join(lines))
 
 
@@ -115,6 +117,9 @@ def draw_tensor(spec, generator: torch.Generator, dtype: torch.dtype, std: float
         t = torch.empty(spec.shape, dtype=f32, device=dev).normal_(0.0, norm_std, generator=generator).to(dtype)
     elif spec.init == "unit_interval":
         t = torch.rand(spec.shape, generator=generator, dtype=f32, device=dev).to(dtype)
+    elif spec.init == "choices":                  # rows of distinct integers below spec.below
+        t = torch.rand((spec.shape[0], spec.below), generator=generator, dtype=f32, device=dev).argsort(dim=1)[:, :spec.shape[1]]
+        t = t.to(torch.int32)
     elif spec.init == "zeros":
         t = torch.zeros(spec.shape, dtype=dtype, device=dev)
     elif spec.init == "a_log":
