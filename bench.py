@@ -245,9 +245,9 @@ def main() -> int:
     ap.add_argument("--no-big", dest="big", action="store_false", help="skip the 3B and 7B workloads among the points")
     ap.add_argument("--no-pairs", action="store_true", help="run the linear layers on single blocks (128 x 256 tiles) instead "
                     "of pairs of blocks on 256 x 256 tiles: the comparison behind profiles/linear_tcgen05_prefill_2048.md")
-    ap.add_argument("--design", default=None, choices=["turevik", "porarax", "sogazen", "kimutar", "kefetar"], help="instead of the benchmark line: prefill and decode "
+    ap.add_argument("--design", default=None, choices=["turevik", "porarax", "sogazen", "kimutar", "kefetar", "fobatar"], help="instead of the benchmark line: prefill and decode "
                     "throughput of this design at layer sizes of a real model's order (random weights), beside the library's "
-                    "closest other design (Falcon-H1 for turevik and sogazen, Turevik for porarax, Porarax for kimutar, Kimutar for kefetar) at equal "
+                    "closest other design (Falcon-H1 for turevik and sogazen, Turevik for porarax, Porarax for kimutar and fobatar, Kimutar for kefetar) at equal "
                     "width and layer count")
     ap.add_argument("--sizes-only", default=None, choices=["width 2048", "width 3072"], help="with --design: one of the two sizes")
     ap.add_argument("--ref-budget", type=float, default=600.0, help="seconds the reference arm may take (it runs fewer "
@@ -572,9 +572,59 @@ def kefetar_work(cfg, batch, context, T):
     return fixed * 2 + cache_bytes, 2.0 * (fixed - V * D) * T + 2.0 * V * D + mix_flops
 
 
+def fobatar_config(width, heads, kv_heads, kv_rank, chunk, experts, top, expert_ff, vocab):
+    """Four layers with both kinds of mixer, experts chosen by token id and a shared expert in each: attention over chunks with
+    convolved and normed projections; latent attention with a rotated part; both again."""
+    rot = lambda dims: dict(base=500000.0, dims=dims, scaling=dict(factor=8.0, original=4096, fast=32.0, slow=1.0))
+    moe = dict(kind="moe", router=dict(experts=experts, top=top), expert=dict(ff=expert_ff, limit=7.0), shared=dict(ff=expert_ff, limit=7.0))
+    att = dict(type="attention", mixer=dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, conv=4, scale=128 ** -0.5, rot=rot(64),
+                                            mask=dict(size=chunk)), mlp=moe)
+    lat = dict(type="latent_attention", mixer=dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=kv_rank, scale=192 ** -0.5,
+                                                   rot=rot(64)), mlp=moe)
+    return dict(architecture="Fobatar", vocab=vocab, width=width, embedding=dict(scale=4.0), norm=dict(eps=1e-6), residual_mult=0.5,
+                layers=[att, lat, att, lat])
+
+
+def porarax_attention_config(width, heads, kv_heads, kv_rank, chunk, experts, top, expert_ff, vocab):
+    """Porarax's layers that are nearest to Fobatar's, at the same sizes and in the same order: attention, latent attention with a
+    latent of its own (queries through a latent of a third of the width, a window wider than the prompt), experts in each."""
+    moe = dict(kind="moe", router=dict(experts=experts, top=top), expert=dict(ff=expert_ff, limit=7.0))
+    att = dict(type="attention", mixer=dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5,
+                                            rot=dict(base=500000.0, dims=64)), mlp=moe)
+    lat = dict(type="latent_attention", mixer=dict(heads=heads, dim=128, vdim=128, kv_rank=kv_rank, q_rank=width // 24 * 8,
+                                                   scale=128 ** -0.5, mask=dict(size=1 << 20)), mlp=moe)
+    return dict(architecture="Porarax", vocab=vocab, width=width, norm=dict(eps=1e-6), layers=[att, lat, att, lat])
+
+
+def fobatar_work(cfg, batch, context, T):
+    """(bytes a decode step of `batch` sequences at `context` must read, FLOPs of a prompt of T tokens)."""
+    D, V = cfg["width"], cfg["vocab"]
+    fixed, cache_bytes, mix_flops, expert_bytes, expert_params = V * D, 0, 0.0, 0.0, 0
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        H, dk, dv = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "attention":
+            G, C = m["kv_heads"], m["mask"]["size"]
+            fixed += (H * dk + G * dk + G * dv + H) * D + D * H * dv
+            cache_bytes += batch * (context % C + 1) * G * (dk + dv) * 2 + batch * (m["conv"] - 1) * (H * dk + G * (dk + dv)) * 4
+            mix_flops += 2.0 * H * (dk + dv) * sum(t % C + 1 for t in range(T))
+        else:
+            R, r = m["kv_rank"], m["rot_dim"]
+            fixed += (H * (dk + r) + R + r + H) * D + H * (dk + dv) * R + D * H * dv
+            cache_bytes += batch * context * (R + r) * 2
+            mix_flops += 2.0 * H * (2 * R + r) * T * (T + 1) / 2           # scores and sums in the latent space
+        mlp = layer["mlp"]
+        E, top, F = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"]
+        fixed += 3 * D * mlp["shared"]["ff"]
+        expert_params += top * 3 * D * F
+        touched = E * (1.0 - (1.0 - top / E) ** batch)                      # expected distinct experts of a step
+        expert_bytes += touched * 3 * D * F * 2
+    return fixed * 2 + expert_bytes + cache_bytes, 2.0 * (fixed - V * D + expert_params) * T + 2.0 * V * D + mix_flops
+
+
 def design_compare(args) -> int:
     """Another design beside the library's closest one at equal width and layer count (Turevik and Sogazen beside Falcon-H1,
-    Porarax beside Turevik, Kimutar beside Porarax, Kefetar beside Kimutar): a prompt of --prefill-tokens tokens and decode steps at batch 8 and 64 from --prompt-len-token
+    Porarax beside Turevik, Kimutar and Fobatar beside Porarax, Kefetar beside Kimutar): a prompt of --prefill-tokens tokens and decode steps at batch 8 and 64 from --prompt-len-token
     prompts, each as time and as a fraction of the measured peak for the bytes a step must read (decode) or the FLOPs a
     prompt needs (prefill)."""
     import torch
@@ -597,6 +647,10 @@ def design_compare(args) -> int:
         sizes_of = {"width 2048": (2048, 16, 4, 4096, 65536), "width 3072": (3072, 24, 8, 12288, 130048)}
         cases = {k: (kefetar_config(*v), kimutar_dense_config(*v)) for k, v in sizes_of.items()}
         beside = "kimutar"
+    elif args.design == "fobatar":
+        sizes_of = {"width 2048": (2048, 16, 4, 256, 1024, 32, 4, 1024, 65536), "width 3072": (3072, 24, 8, 256, 1024, 64, 6, 2048, 130048)}
+        cases = {k: (fobatar_config(*v), porarax_attention_config(*v)) for k, v in sizes_of.items()}
+        beside = "porarax"
     elif args.design == "sogazen":
         cases = {"width 2048": (sogazen_config(2048, 8, 2, 48, 64, 256, 32, 4096, 32, 4, 4, 1024, 65536), dict(CONFIG_1P5B, num_hidden_layers=4)),
                  "width 3072": (sogazen_config(3072, 12, 2, 24, 128, 256, 48, 12288, 64, 8, 6, 2048, 130048), dict(CONFIG_7B, num_hidden_layers=4))}
@@ -606,7 +660,7 @@ def design_compare(args) -> int:
                  "width 3072": (turevik["width 3072"], dict(CONFIG_7B, num_hidden_layers=4))}
         beside = "falcon_h1"
     work = {"turevik": turevik_work, "porarax": porarax_work, "sogazen": sogazen_work, "kimutar": kimutar_work,
-            "kefetar": kefetar_work}
+            "kefetar": kefetar_work, "fobatar": fobatar_work}
     if args.sizes_only:
         cases = {k: v for k, v in cases.items() if k == args.sizes_only}
     for name, (tcfg, fcfg) in cases.items():

@@ -419,3 +419,85 @@ def kefetar_random(seed: int) -> dict:
                                pick(None, 2.0, 10.0), v_mix, _kef_rot(base, dims, pick(None, 1.5, 4.0)), ff))
     return dict(architecture="Kefetar", vocab=pick(50, 131, 300), width=pick(32, 44, 50, 64, 96), norm=dict(eps=pick(1e-5, 1e-6)),
                 canon=dict(taps=pick(1, 2, 3, 4, 6)), layers=layers)
+
+
+# ---- Fobatar ------------------------------------------------------------------------------------------------------------------
+def _fob_att(heads, kv_heads, dim, vdim, conv, scale, rot, chunk, mlp):
+    m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, conv=conv, scale=scale, rot=rot)
+    if chunk:
+        m["mask"] = dict(size=chunk)
+    return dict(type="attention", mixer=m, mlp=mlp)
+
+
+def _fob_lat(heads, dim, rot_dim, vdim, kv_rank, scale, rot, mlp):
+    return dict(type="latent_attention", mixer=dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, scale=scale, rot=rot),
+                mlp=mlp)
+
+
+def _fob_moe(experts, top, ff, limit, shared=None):
+    mlp = dict(kind="moe", router=dict(experts=experts, top=top), expert=dict(ff=ff, limit=limit))
+    if shared:
+        mlp["shared"] = dict(ff=shared[0], limit=shared[1])
+    return mlp
+
+
+# A: the repeated range from layer 0, three times; a width and feed-forwards that are no multiples of 8; chunks of 5 and of 70
+# positions and none; keys wider and narrower than values, one head per key head, six on one, two, four and one taps; a ramp, plain
+# frequencies and no rotation at all; latents of 20 and 33 values (no tensor-core kernel), two thirds of the rotated part
+# rotated; every expert chosen, a single expert, one chosen of five; with and without a shared expert; a layer without
+# feed-forward
+FOBATAR_A = dict(architecture="Fobatar", vocab=150, width=52, embedding=dict(scale=3.0), norm=dict(eps=1e-5), residual_mult=0.6,
+                 loop=dict(start=0, stop=2, times=3), layers=[
+    _fob_att(4, 2, 24, 16, 2, 0.3, _k_rot(100.0, 8, factor=4.0, original=64, fast=8.0, slow=2.0), 5, _fob_moe(4, 2, 20, 1.0, shared=(12, 0.7))),
+    _fob_lat(3, 10, 6, 14, 20, 0.25, _k_rot(10000.0, 4), None),
+    _fob_att(6, 1, 20, 32, 4, 0.2, _k_rot(500.0, 20, factor=2.0, original=100, fast=16.0, slow=1.0), 70, _fob_moe(3, 3, 16, 0.5)),
+    _fob_att(2, 2, 16, 16, 1, 0.25, _k_rot(10000.0, 0), None, _fob_moe(1, 1, 24, 2.0, shared=(24, 0.4))),
+    _fob_lat(5, 8, 8, 8, 33, 0.3, _k_rot(300.0, 8, factor=8.0, original=50, fast=4.0, slow=1.0), _fob_moe(5, 1, 12, 1.5, shared=(20, 1.0))),
+])
+
+# B: heads of 64 and of 128 (the tcgen05 attention of prompts, the one-kernel attention of single tokens) in chunks of 100, of
+# 33 and of exactly a page, values narrower than keys, three to five taps; latents of 48 and 80 values behind rotated parts of 16
+# and 32 (the tensor-core kernel); the repeated range in the middle, twice; latent attention first
+FOBATAR_B = dict(architecture="Fobatar", vocab=97, width=64, embedding=dict(scale=5.0), norm=dict(eps=1e-6), residual_mult=0.8,
+                 loop=dict(start=1, stop=3, times=2), layers=[
+    _fob_lat(4, 16, 16, 24, 48, 0.18, _k_rot(10000.0, 16, factor=4.0, original=64, fast=8.0, slow=1.0), _fob_moe(6, 2, 32, 1.0, shared=(16, 2.0))),
+    _fob_att(4, 2, 64, 64, 3, 0.11, _k_rot(50000.0, 32, factor=2.0, original=100, fast=16.0, slow=1.0), 100,
+             _fob_moe(8, 3, 24, 0.8, shared=(40, 1.2))),
+    _fob_att(2, 1, 128, 128, 4, 0.07, _k_rot(1000000.0, 128, factor=8.0, original=128, fast=32.0, slow=1.0), 33, None),
+    _fob_lat(2, 32, 32, 16, 80, 0.15, _k_rot(700.0, 32), _fob_moe(4, 2, 16, 1.0)),
+    _fob_att(2, 2, 64, 40, 5, 0.12, _k_rot(300.0, 16), 64, _fob_moe(2, 1, 40, 1.0)),
+])
+
+FOBATAR = {"OA": FOBATAR_A, "OB": FOBATAR_B}
+
+
+def fobatar_random(seed: int) -> dict:
+    """A Fobatar configuration drawn from `seed`: 2 to 5 layers of both kinds in any order, a repeated range or none, with head
+    counts, sizes, rotated dimensions, scalings, chunks, taps, experts, limits and constants all drawn."""
+    import numpy as np
+    rng = np.random.default_rng(seed)
+    pick = lambda *v: v[int(rng.integers(len(v)))]
+    layers = []
+    for _ in range(int(rng.integers(2, 6))):
+        mlp = None
+        if rng.random() < 0.8:
+            experts = pick(1, 2, 3, 5, 8, 40)
+            mlp = _fob_moe(experts, int(rng.integers(1, min(experts, 4) + 1)), pick(8, 12, 24, 40), pick(0.4, 1.0, 7.0),
+                           shared=pick(None, (8, 0.5), (20, 3.0)))
+        sc = pick(None, dict(factor=pick(2.0, 6.0), original=pick(32, 100), fast=pick(8.0, 32.0), slow=pick(1.0, 2.0)))
+        base = pick(50.0, 10000.0, 500000.0)
+        if rng.random() < 0.5:
+            rot_dim = pick(2, 6, 8, 16, 32)
+            dim = pick(4, 8, 10, 16, 32)
+            layers.append(_fob_lat(pick(1, 2, 3, 5), dim, rot_dim, pick(4, 8, 14, 16, 24), pick(12, 16, 32, 33, 48),
+                                   float((dim + rot_dim) ** -0.5 * rng.uniform(0.5, 2.0)), _k_rot(base, pick(rot_dim, rot_dim, 2), **(sc or {})), mlp))
+            continue
+        kv, dim = pick(1, 2, 3), pick(8, 10, 16, 24, 64, 128)
+        layers.append(_fob_att(kv * pick(1, 2, 3, 5), kv, dim, pick(6, 8, 16, 20, 64), pick(1, 2, 3, 4, 6), float(dim ** -0.5 * rng.uniform(0.5, 2.0)),
+                               _k_rot(base, pick(0, 2, dim // 4 * 2, dim), **(sc or {})), pick(None, 1, 7, 40, 64, 90), mlp))
+    cfg = dict(architecture="Fobatar", vocab=pick(50, 131, 300), width=pick(32, 44, 50, 64, 96), embedding=dict(scale=pick(1.0, 2.5, 8.0)),
+               norm=dict(eps=pick(1e-5, 1e-6)), residual_mult=pick(0.5, 1.0, 1.3), layers=layers)
+    if rng.random() < 0.7:
+        start = int(rng.integers(0, len(layers)))
+        cfg["loop"] = dict(start=start, stop=int(rng.integers(start + 1, len(layers) + 1)), times=pick(1, 2, 3))
+    return cfg

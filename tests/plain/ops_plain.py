@@ -140,19 +140,18 @@ def attention(q, k_pages, v_pages, block_table, positions, row_seq, slots, out, 
         pages = table[(idx // PAGE).long()].long()
         K = _f(k_pages[pages, :, (idx % PAGE).long(), :])          # [n, KV, hd]
         V = _f(v_pages[pages, :, (idx % PAGE).long(), :])
-        for h in range(H):
-            g = h // (H // KV)
-            sc = (K[:, g] @ qf[t, h]) * scale
-            if softcap:
-                sc = softcap * torch.tanh(sc / softcap)
-            if sink or sink_values is not None:   # one more term (score 0, or the head's own) in the denominator, with no value
-                sv = sc.new_zeros(1) if sink_values is None else _f(sink_values[h]).reshape(1)
-                pr = torch.softmax(torch.cat([sc, sv]), dim=0)[:-1]
-            else:
-                pr = torch.softmax(sc, dim=0)
-            res[t, h] = pr @ V[:, g]
-            if head_gate is not None:
-                res[t, h] *= 1.0 / (1.0 + torch.exp(-_f(head_gate[t, h])))
+        # scores of all heads, head h on key/value head h // (H // KV): [KV, H // KV, n]
+        sc = torch.einsum("grd,ngd->grn", qf[t].reshape(KV, H // KV, hd), K) * scale
+        if softcap:
+            sc = softcap * torch.tanh(sc / softcap)
+        if sink or sink_values is not None:   # one more term (score 0, or the head's own) in the denominator, with no value
+            sv = sc.new_zeros(H) if sink_values is None else _f(sink_values)
+            pr = torch.softmax(torch.cat([sc, sv.reshape(KV, H // KV, 1)], dim=2), dim=2)[:, :, :-1]
+        else:
+            pr = torch.softmax(sc, dim=2)
+        res[t] = torch.einsum("grn,ngd->grd", pr, V).reshape(H, hd)
+        if head_gate is not None:
+            res[t] *= (1.0 / (1.0 + torch.exp(-_f(head_gate[t])))).unsqueeze(1)
     out.copy_(res.reshape(T, H * hd).to(out.dtype))
 
 
