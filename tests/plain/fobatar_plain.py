@@ -88,8 +88,10 @@ def rotate_neighbours(x, pos, freq, grow):
 
 # ---- attention ----------------------------------------------------------------------------------------------------------
 def visible(i, j, chunk=None):
-    """Whether query position i sees key position j: causal, and with a chunk size only within i's chunk."""
-    return j <= i and (chunk is None or i // chunk == j // chunk)
+    """Whether query position i sees key position j (a number or an array of them): causal, and with a chunk size only within
+    i's chunk."""
+    seen = j <= i
+    return seen if chunk is None else seen & (i // chunk == j // chunk)
 
 
 def attend(q, k, v, scale, chunk=None, sink=False):
@@ -97,7 +99,7 @@ def attend(q, k, v, scale, chunk=None, sink=False):
     T = q.shape[0]
     out = np.zeros((T, v.shape[1]))
     for i in range(T):
-        js = [j for j in range(i + 1) if visible(i, j, chunk)]
+        js = np.flatnonzero(visible(i, np.arange(T), chunk))
         s = (k[js] @ q[i]) * scale
         top = max(s.max(), 0.0) if sink else s.max()
         e = np.exp(s - top)

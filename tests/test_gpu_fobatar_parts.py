@@ -221,15 +221,17 @@ def _round_all(W):
 RAMP = dict(factor=4.0, original=64, fast=8.0, slow=1.0)
 
 
+@pytest.mark.parametrize("at_once", [True, False])
 @pytest.mark.parametrize("dtype", list(DT))
 @pytest.mark.parametrize("H,KV,dim,vdim,taps,rot,chunk", [
     (4, 2, 24, 16, 3, dict(base=100.0, dims=8, scaling=RAMP), 37), (3, 1, 16, 20, 1, dict(base=5000.0, dims=16), 5),
     (4, 2, 64, 64, 4, dict(base=10000.0, dims=32, scaling=RAMP), 100), (2, 2, 128, 128, 2, dict(base=700.0, dims=128, scaling=RAMP), 64),
     (6, 2, 64, 48, 5, dict(base=700.0, dims=0), None), (3, 3, 40, 64, 4, dict(base=900.0, dims=20, scaling=RAMP), 150),
     (9, 1, 128, 64, 4, dict(base=900.0, dims=6), 33)])
-def test_chunked_attention_mixer_over_schedules(dtype, H, KV, dim, vdim, taps, rot, chunk):
-    """The whole mixer: the oldest tap speaks loudest and one row is loud, so an echo one row short or long shows; the sharp
+def test_chunked_attention_mixer_over_schedules(monkeypatch, dtype, H, KV, dim, vdim, taps, rot, chunk, at_once):
+    """The whole mixer, with convolution, norm, rotation and stores in one kernel and in kernels of their own: the oldest tap speaks loudest and one row is loud, so an echo one row short or long shows; the sharp
     score scale makes single keys decide."""
+    monkeypatch.setattr(ops, "DISABLE_QKV_PREPARE", not at_once)
     D, eps = 40, 1e-5
     g = np.random.default_rng(H * 100 + dim)
     W = {"q": g.standard_normal((H * dim, D)), "k": g.standard_normal((KV * dim, D)), "v": g.standard_normal((KV * vdim, D)),
@@ -299,13 +301,19 @@ def test_latent_attention_mixer_over_schedules(dtype, H, dim, r, vdim, R, rot):
 
 
 # ---- experts chosen by a table --------------------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("V,E,top,T", [(50, 4, 2, 1), (50, 4, 4, 33), (1000, 40, 3, 300), (7, 1, 1, 9), (300, 100, 7, 2049)])
+@pytest.mark.parametrize("V,E,top,T", [(50, 4, 2, 1), (50, 4, 4, 33), (1000, 40, 3, 300), (7, 1, 1, 9), (300, 100, 7, 2049), (90, 32, 5, 500)])
 def test_routing_by_a_table(V, E, top, T):
     g = np.random.default_rng(E)
     table = np.stack([g.permutation(E)[:top] for _ in range(V)]).astype(np.int32)
     toks = g.integers(0, V, T).astype(np.int32)
     for tile in (32, 64):
-        ids, wts, order, offsets, tile_off, rows = ops.moe_route_table(dev(toks, torch.int32), dev(table, torch.int32), E, 1.0 / top, tile)
+        # between two other tables: every one of a launch has ranges of its own
+        others = [(dev(table[:, :1], torch.int32), E, False), (dev(np.tile(np.arange(2), (V, 1)), torch.int32), 2, True)]
+        tables = ops.ExpertTables([others[0], (dev(table, torch.int32), E, tile == 64), others[1]])
+        tile = 64 if tile == 64 and T * top >= 64 * E else 32
+        routed = ops.moe_route_tables(dev(toks, torch.int32), tables)
+        assert np.array_equal(routed[0][0].cpu().numpy(), table[toks][:, 0]) and np.array_equal(routed[2][0].cpu().numpy(), np.tile([0, 1], T))
+        ids, wts, order, offsets, tile_off, rows = routed[1]
         want = table[toks].reshape(-1)
         assert np.array_equal(ids.cpu().numpy(), want) and rows == tile
         assert np.allclose(wts.cpu().numpy(), 1.0 / top)
@@ -343,10 +351,16 @@ def test_experts_of_a_table_with_both_clamps_at_work(dtype, D, F, E, top, shared
     for T in (1, 5, 40, 130, 400):
         x, toks = plain.bf16_round(g.standard_normal((T, D)) * 2.0), g.integers(0, V, T)
         out = torch.full((T, D), 5.0, device="cuda")
-        ff.forward(dev(x, DT[dtype]), out, accumulate=False, tokens=dev(toks, torch.int32))
+        step = type("Step", (), dict(tokens=dev(toks, torch.int32), scratch={}))
+        ff.forward(dev(x, DT[dtype]), out, accumulate=False, step=step)
         want = plain.table_moe(x, toks, W, p, mlp)
         tol = 3e-5 if dtype == "float32" else 1.2e-2
         assert np.abs(out.cpu().numpy() - want).max() <= tol * np.abs(want).max(), f"{T} rows"
+        before = out.clone()
+        ff.route_step([ff], ops.ExpertTables([ff.table_entry()]), step)       # the routing made ahead of the layers is the same
+        out.fill_(5.0)
+        ff.forward(dev(x, DT[dtype]), out, accumulate=False, step=step)
+        assert torch.equal(before, out)
     with pytest.raises(ValueError, match="token ids"):
         ff.forward(dev(x, DT[dtype]), out)
 
@@ -376,6 +390,25 @@ def test_embedding_added_to_the_stream(dtype, D):
     assert np.abs(xd.cpu().numpy() - want).max() <= 1e-6 * np.abs(want).max()
     ops.embed(dev(toks, torch.int32), dev(table, DT[dtype]), 1.7, first)
     assert np.abs(first.cpu().numpy() - table[toks] * 1.7).max() <= 1e-6 * np.abs(table).max()
+
+
+@pytest.mark.parametrize("dtype", list(DT))
+@pytest.mark.parametrize("D,T", [(5, 3), (52, 9), (64, 300), (2048, 8), (2048, 1500), (4098, 4)])
+def test_output_norm_that_leaves_the_next_norm_of_the_stream(dtype, D, T):
+    """One kernel adds a normed result (a sum of terms) into the stream and norms the new rows for the sublayer that follows."""
+    g = np.random.default_rng(D)
+    w, w2 = 1 + 0.2 * g.standard_normal(D), 1 + 0.2 * g.standard_normal(D)
+    parts, extra, x = g.standard_normal((T, 3, D)), g.standard_normal((T, D)), g.standard_normal((T, D)) * 0.01
+    make = lambda name, weight, scale: PartSpec("norm", "rmsnorm", dict(width=D, eps=1e-5, weight_name=name, scale=scale)).build()
+    norm, nxt = make("w", w, 0.003), make("v", w2, 1.0)                # (a stream so small that eps matters)
+    for n, v in ((norm, w), (nxt, w2)):
+        n.bind({"w": torch.tensor(v), "v": torch.tensor(v)}, torch.float32, torch.device("cuda"))
+    xd, left = dev(x), torch.full((T, D), 7.0, dtype=DT[dtype], device="cuda")
+    norm.add_normed(dev(parts), xd, dev(extra), None, copy=left, next_norm=nxt)
+    want = x + 0.003 * plain.rms_norm(parts.sum(1) + extra, w, 1e-5)
+    assert np.abs(xd.cpu().numpy() - want).max() <= 2e-5 * np.abs(want).max()
+    want = plain.rms_norm(want, w2, 1e-5)
+    assert np.abs(left.float().cpu().numpy() - want).max() <= (3e-5 if dtype == "float32" else 5e-3) * np.abs(want).max()
 
 
 def test_norm_with_a_multiplier_adds_into_the_stream():

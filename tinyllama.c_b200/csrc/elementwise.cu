@@ -21,38 +21,17 @@ int tlc_fail(int code, const char* fmt, ...) {
 }
 
 // ---- embedding ---------------------------------------------------------------------
-template <typename TW>
-__global__ void embed_kernel(const int* __restrict__ tokens, const TW* __restrict__ table, int D, int V,
-                             float scale, float* __restrict__ out) {
+// out[t] = table[tokens[t]] * scale, or with ADD out[t] += it (a pass of a repeated range of layers begins with the embedding
+// once more).  Four values a thread where rows lie on 16-byte (bfloat16: 8-byte) boundaries.
+template <typename TW, int VEC, bool ADD>
+__global__ void __launch_bounds__(256)
+embed_kernel(const int* __restrict__ tokens, const TW* __restrict__ table, int D, int V, float scale, float* __restrict__ out) {
   tlc_pdl(tokens, out);
   const int t = blockIdx.x;
   int tok = tokens[t];
   tok = tok < 0 ? 0 : (tok >= V ? V - 1 : tok);   // ids are validated on the host; never read out of bounds
   const TW* row = table + (size_t)tok * D;
-  for (int d = threadIdx.x; d < D; d += blockDim.x) out[(size_t)t * D + d] = to_f32(row[d]) * scale;
-}
-
-extern "C" int tlc_embed(const int* tokens, const void* table, int table_dtype, int T, int D, int V, float scale,
-                         float* out, cudaStream_t stream) {
-  if (T == 0) return 0;
-  // the first kernel of a step: a full dependency on everything before it (see tlc_launch_step_boundary)
-  TLC_DISPATCH_DTYPE(table_dtype, TW, tlc_launch_step_boundary(embed_kernel<TW>, dim3(T), dim3(256), 0, stream, tokens,
-                                                               (const TW*)table, D, V, scale, out));
-  TLC_CHECK_LAUNCH("embed");
-  return 0;
-}
-
-// x[t] += table[tokens[t]] * scale: the embedding once more (a pass of a repeated range of layers begins with it).  Four
-// values a thread where rows lie on 16-byte (8-byte) boundaries.
-template <typename TW, int VEC>
-__global__ void __launch_bounds__(256)
-embed_add_kernel(const int* __restrict__ tokens, const TW* __restrict__ table, int D, int V, float scale, float* __restrict__ x) {
-  tlc_pdl(x);
-  const int t = blockIdx.x;
-  int tok = tokens[t];
-  tok = tok < 0 ? 0 : (tok >= V ? V - 1 : tok);
-  const TW* row = table + (size_t)tok * D;
-  float* xr = x + (size_t)t * D;
+  float* o = out + (size_t)t * D;
   for (int d = threadIdx.x * VEC; d < D; d += blockDim.x * VEC) {
     if (VEC == 4) {
       float4 e;
@@ -63,25 +42,38 @@ embed_add_kernel(const int* __restrict__ tokens, const TW* __restrict__ table, i
       } else {
         e = *reinterpret_cast<const float4*>(row + d);
       }
-      float4 v = *reinterpret_cast<const float4*>(xr + d);
-      v.x = fmaf(e.x, scale, v.x); v.y = fmaf(e.y, scale, v.y); v.z = fmaf(e.z, scale, v.z); v.w = fmaf(e.w, scale, v.w);
-      *reinterpret_cast<float4*>(xr + d) = v;
+      float4 v = ADD ? *reinterpret_cast<const float4*>(o + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+      if (ADD) { v.x = fmaf(e.x, scale, v.x); v.y = fmaf(e.y, scale, v.y); v.z = fmaf(e.z, scale, v.z); v.w = fmaf(e.w, scale, v.w); }
+      else v = make_float4(e.x * scale, e.y * scale, e.z * scale, e.w * scale);
+      *reinterpret_cast<float4*>(o + d) = v;
     } else {
-      xr[d] = fmaf(to_f32(row[d]), scale, xr[d]);
+      o[d] = ADD ? fmaf(to_f32(row[d]), scale, o[d]) : to_f32(row[d]) * scale;
     }
   }
 }
 
+template <bool ADD>
+static int embed_launch(const int* tokens, const void* table, int table_dtype, int T, int D, int V, float scale, float* out,
+                        cudaStream_t stream) {
+  if (T == 0) return 0;
+  const bool vec = D % 4 == 0 && (uintptr_t)table % 16 == 0 && (uintptr_t)out % 16 == 0;
+  // the first kernel of a step: a full dependency on everything before it (see tlc_launch_step_boundary)
+  TLC_DISPATCH_DTYPE(table_dtype, TW, {
+    if (vec) tlc_launch_as(ADD, embed_kernel<TW, 4, ADD>, dim3(T), dim3(256), 0, stream, tokens, (const TW*)table, D, V, scale, out);
+    else tlc_launch_as(ADD, embed_kernel<TW, 1, ADD>, dim3(T), dim3(256), 0, stream, tokens, (const TW*)table, D, V, scale, out);
+  });
+  TLC_CHECK_LAUNCH("embed");
+  return 0;
+}
+
+extern "C" int tlc_embed(const int* tokens, const void* table, int table_dtype, int T, int D, int V, float scale, float* out,
+                         cudaStream_t stream) {
+  return embed_launch<false>(tokens, table, table_dtype, T, D, V, scale, out, stream);
+}
+
 extern "C" int tlc_embed_add(const int* tokens, const void* table, int table_dtype, int T, int D, int V, float scale, float* x,
                              cudaStream_t stream) {
-  if (T == 0) return 0;
-  const bool vec = D % 4 == 0 && (uintptr_t)table % 16 == 0 && (uintptr_t)x % 16 == 0;
-  TLC_DISPATCH_DTYPE(table_dtype, TW, {
-    if (vec) tlc_launch(embed_add_kernel<TW, 4>, dim3(T), dim3(256), 0, stream, tokens, (const TW*)table, D, V, scale, x);
-    else tlc_launch(embed_add_kernel<TW, 1>, dim3(T), dim3(256), 0, stream, tokens, (const TW*)table, D, V, scale, x);
-  });
-  TLC_CHECK_LAUNCH("embed_add");
-  return 0;
+  return embed_launch<true>(tokens, table, table_dtype, T, D, V, scale, x, stream);
 }
 
 // ---- RMSNorm of 32-bit rows ----------------------------------------------------------
@@ -525,7 +517,8 @@ extern "C" int tlc_rmsnorm_shift(const float* x, const float* w, const float* mu
 __global__ void __launch_bounds__(1024)
 rmsnorm_add_kernel(const float* __restrict__ parts, int n_parts, const float* __restrict__ extra,
                    const float* __restrict__ gate, int gate_ld, int gate_sigmoid, const float* __restrict__ w, float eps, int D,
-                   float* __restrict__ res, int accumulate, int keep, void* __restrict__ copy, int copy_dtype) {
+                   float* __restrict__ res, int accumulate, int keep, void* __restrict__ copy, int copy_dtype,
+                   const float* __restrict__ next_w, float next_eps) {
   tlc_pdl(parts, extra, gate, res, copy);
   __shared__ float red[33];
   extern __shared__ float yrow[];               // the summed row, where it fits (keep)
@@ -564,8 +557,13 @@ rmsnorm_add_kernel(const float* __restrict__ parts, int n_parts, const float* __
     float* o = res + (size_t)t * D + d;
     const float r = accumulate ? *o + v : v;
     *o = r;
-    if (copy) put_as(copy, copy_dtype, (size_t)t * D + d, r);
+    if (copy && !next_w) put_as(copy, copy_dtype, (size_t)t * D + d, r);
   }
+  if (!copy || !next_w) return;
+  float n2 = 0.f;                               // the copy is the new row, normed for the sublayer that follows
+  for (int d = threadIdx.x; d < D; d += blockDim.x) { const float r = res[(size_t)t * D + d]; n2 += r * r; }     // (this thread's own)
+  const float ns = 1.0f / sqrtf(block_sum(n2, red) / (float)D + next_eps);
+  for (int d = threadIdx.x; d < D; d += blockDim.x) put_as(copy, copy_dtype, (size_t)t * D + d, res[(size_t)t * D + d] * ns * next_w[d]);
 }
 
 // The same with a row in registers: 16-byte loads and stores, the weight fetched before the wait on the previous kernel.
@@ -574,7 +572,8 @@ template <int NT, int PT>
 __global__ void __launch_bounds__(NT)
 rmsnorm_add_vec_kernel(const float* __restrict__ parts, int n_parts, const float* __restrict__ extra,
                        const float* __restrict__ gate, int gate_ld, int gate_sigmoid, const float* __restrict__ w, float eps,
-                       int D, float* __restrict__ res, int accumulate, void* __restrict__ copy, int copy_dtype) {
+                       int D, float* __restrict__ res, int accumulate, void* __restrict__ copy, int copy_dtype,
+                       const float* __restrict__ next_w, float next_eps) {
   asm volatile("griddepcontrol.launch_dependents;");
   __shared__ float red[33];
   const int n4 = D >> 2, t = blockIdx.x;
@@ -638,7 +637,25 @@ rmsnorm_add_vec_kernel(const float* __restrict__ parts, int n_parts, const float
       r[i].x += v[i].x; r[i].y += v[i].y; r[i].z += v[i].z; r[i].w += v[i].w;
     }
     rr[c] = r[i];
-    if (copy) put4_as(copy, copy_dtype, (size_t)t * D + 4 * c, r[i]);
+    if (copy && !next_w) put4_as(copy, copy_dtype, (size_t)t * D + 4 * c, r[i]);
+  }
+  if (!copy || !next_w) return;
+  float n2 = 0.f;                                          // the copy is the new row, normed for the sublayer that follows
+#pragma unroll
+  for (int i = 0; i < PT; i++) {
+    const int c = threadIdx.x + i * NT;
+    if (c < n4) {
+      n2 += r[i].x * r[i].x + r[i].y * r[i].y + r[i].z * r[i].z + r[i].w * r[i].w;
+      wv[i] = __ldg(reinterpret_cast<const float4*>(next_w) + c);       // (in flight during the block's sum)
+    }
+  }
+  const float ns = 1.0f / sqrtf(block_sum(n2, red) / (float)D + next_eps);
+#pragma unroll
+  for (int i = 0; i < PT; i++) {
+    const int c = threadIdx.x + i * NT;
+    if (c < n4)
+      put4_as(copy, copy_dtype, (size_t)t * D + 4 * c,
+              make_float4(r[i].x * ns * wv[i].x, r[i].y * ns * wv[i].y, r[i].z * ns * wv[i].z, r[i].w * ns * wv[i].w));
   }
 }
 
@@ -646,15 +663,15 @@ static bool aligned16(const void* p) { return ((uintptr_t)p % 16) == 0; }
 
 extern "C" int tlc_rmsnorm_add(const float* parts, int n_parts, const float* extra, const float* gate, int gate_ld,
                                int gate_sigmoid, const float* w, float eps, int T, int D, float* res, int accumulate,
-                               void* copy, int copy_dtype, cudaStream_t stream) {
+                               void* copy, int copy_dtype, const float* next_w, float next_eps, cudaStream_t stream) {
   if (T == 0) return 0;
   TLC_REQUIRE(n_parts >= 0 && (n_parts > 0 || extra != nullptr), "rmsnorm_add: nothing to add");
   TLC_REQUIRE(copy == nullptr || copy_dtype == TLC_F32 || copy_dtype == TLC_BF16, "rmsnorm_add: unknown dtype code %d of the copy", copy_dtype);
-  if (D % 4 == 0 && D <= 16384 && aligned16(parts) && aligned16(extra) && aligned16(w) && aligned16(res) && aligned16(copy)) {
+  if (D % 4 == 0 && D <= 16384 && aligned16(parts) && aligned16(extra) && aligned16(w) && aligned16(res) && aligned16(copy) && aligned16(next_w)) {
     const int n4 = D / 4;
 #define TLC_RA_LAUNCH(NT, PT)                                                                                             \
   tlc_launch(rmsnorm_add_vec_kernel<NT, PT>, dim3(T), dim3(NT), 0, stream, parts, n_parts, extra, gate, gate_ld, gate_sigmoid, w, \
-             eps, D, res, accumulate, copy, copy_dtype)
+             eps, D, res, accumulate, copy, copy_dtype, next_w, next_eps)
     if (T >= VEC_MANY_ROWS) { TLC_VEC_SHAPES_MANY(n4, TLC_RA_LAUNCH) } else { TLC_VEC_SHAPES(n4, TLC_RA_LAUNCH) }
 #undef TLC_RA_LAUNCH
     TLC_CHECK_LAUNCH("rmsnorm_add");
@@ -664,7 +681,7 @@ extern "C" int tlc_rmsnorm_add(const float* parts, int n_parts, const float* ext
   // few rows (single-token steps): more threads a row, so that a thread's loads are few and in flight together
   const int nt = (T < 256 && D >= 1024) ? 1024 : 256;
   tlc_launch(rmsnorm_add_kernel, dim3(T), dim3(nt), keep ? (size_t)D * sizeof(float) : 0, stream, parts, n_parts, extra, gate, gate_ld,
-             gate_sigmoid, w, eps, D, res, accumulate, keep, copy, copy_dtype);
+             gate_sigmoid, w, eps, D, res, accumulate, keep, copy, copy_dtype, next_w, next_eps);
   TLC_CHECK_LAUNCH("rmsnorm_add");
   return 0;
 }

@@ -84,6 +84,85 @@ latent_prepare_kernel(const float* __restrict__ qproj, int ldq, int q_off, const
   }
 }
 
+// The same four neighbouring values a thread (sizes, strides and offsets that are multiples of 4): the row's cosines and sines
+// are computed once and shared by all heads, and the latent is read before the query parts, so that its sum of squares forms
+// while they travel.
+__device__ __forceinline__ void lp_put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void lp_put4(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<const unsigned*>(&lo);
+  u.y = *reinterpret_cast<const unsigned*>(&hi);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+// pairs d, d+1 and d+2, d+3 of a rotated part; cs: [half] cosines | [half] sines
+__device__ __forceinline__ float4 lp_turn4(float4 y, int d, int rot, const float* cs) {
+  const int half = rot >> 1, p = d >> 1;
+  if (d < rot) {
+    const float c = cs[p], s = cs[half + p], u = y.x, v = y.y;
+    y.x = u * c - v * s;
+    y.y = v * c + u * s;
+  }
+  if (d + 2 < rot) {
+    const float c = cs[p + 1], s = cs[half + p + 1], u = y.z, v = y.w;
+    y.z = u * c - v * s;
+    y.w = v * c + u * s;
+  }
+  return y;
+}
+template <typename TC>
+__global__ void __launch_bounds__(512)
+latent_prepare_vec_kernel(const float* __restrict__ qproj, int ldq, int q_off, const float* __restrict__ proj, int ld, int dkv_off,
+                          const float* __restrict__ cw, float eps, const float* __restrict__ inv_freq, int rot,
+                          const int* __restrict__ positions, const int* __restrict__ row_seq, const int* __restrict__ slots,
+                          const int* __restrict__ block_table, int max_pages, TC* __restrict__ pages, TC* __restrict__ qn,
+                          TC* __restrict__ qa, int H, int dn, int r, int R, float amplitude) {
+  asm volatile("griddepcontrol.launch_dependents;");
+  __shared__ float red[33];
+  extern __shared__ float cs[];                            // [rot]
+  const int t = blockIdx.x, pos = positions[t], half = rot >> 1;
+  for (int j = threadIdx.x; j < half; j += blockDim.x) {
+    float sn, c;
+    sincosf((float)pos * inv_freq[j], &sn, &c);
+    cs[j] = c * amplitude;
+    cs[half + j] = sn * amplitude;
+  }
+  const int page = dkv_off < 0 ? 0 : block_table[(size_t)slots[row_seq[t]] * max_pages + pos / TLC_PAGE];
+  tlc_wait(qproj, proj, pages, qn, qa);
+  __syncthreads();
+  const float* pr = qproj + (size_t)t * ldq + q_off;
+  const float* cr = proj + (size_t)t * ld + dkv_off;       // (not read where there is none)
+  const int hw = dn + r, aw = R + r, R4 = R >> 2, r4 = r >> 2, d4 = dn >> 2;
+  float4 c0 = make_float4(0.f, 0.f, 0.f, 0.f);             // a thread's first group of the latent stays in registers
+  float ss = 0.f;
+  if (dkv_off >= 0) {
+    if (threadIdx.x < R4) c0 = *reinterpret_cast<const float4*>(cr + 4 * threadIdx.x);
+    ss = c0.x * c0.x + c0.y * c0.y + c0.z * c0.z + c0.w * c0.w;
+    for (int i = threadIdx.x + blockDim.x; i < R4; i += blockDim.x) {
+      const float4 c = *reinterpret_cast<const float4*>(cr + 4 * i);
+      ss += c.x * c.x + c.y * c.y + c.z * c.z + c.w * c.w;
+    }
+  }
+  const int per = d4 + r4;                                 // groups of a head: its unrotated part, its rotated one
+#pragma unroll 4
+  for (int i = threadIdx.x; i < H * per; i += blockDim.x) {
+    const int h = i / per, j = i - h * per;
+    const float4 v = *reinterpret_cast<const float4*>(pr + (size_t)h * hw + 4 * j);
+    if (j < d4) lp_put4(qn + ((size_t)t * H + h) * dn + 4 * j, v);
+    else lp_put4(qa + ((size_t)t * H + h) * aw + R + 4 * (j - d4), lp_turn4(v, 4 * (j - d4), rot, cs));
+  }
+  if (dkv_off < 0) return;
+  const float s = 1.0f / sqrtf(block_sum(ss, red) / (float)R + eps);
+  TC* row = pages + ((size_t)page * TLC_PAGE + pos % TLC_PAGE) * aw;
+  for (int i = threadIdx.x; i < R4; i += blockDim.x) {
+    const float4 c = i == threadIdx.x ? c0 : *reinterpret_cast<const float4*>(cr + 4 * i);
+    const float4 w = *reinterpret_cast<const float4*>(cw + 4 * i);
+    lp_put4(row + 4 * i, make_float4(c.x * s * w.x, c.y * s * w.y, c.z * s * w.z, c.w * s * w.w));
+  }
+  for (int j = threadIdx.x; j < r4; j += blockDim.x)
+    lp_put4(row + R + 4 * j, lp_turn4(*reinterpret_cast<const float4*>(cr + R + 4 * j), 4 * j, rot, cs));
+}
+
 extern "C" int tlc_latent_prepare(const float* qproj, int ldq, int q_off, const float* proj, int ld, int dkv_off, const float* cw,
                                   float eps,
                                   const float* inv_freq, int rot, const int* positions, const int* row_seq, const int* slots,
@@ -92,6 +171,14 @@ extern "C" int tlc_latent_prepare(const float* qproj, int ldq, int q_off, const 
   if (T == 0) return 0;
   TLC_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= r, "latent_prepare: %d rotated dimensions of %d", rot, r);
   const int nt = T < 256 ? 512 : 128;                       // few rows: more threads a row
+  if (dn % 4 == 0 && r % 4 == 0 && R % 4 == 0 && ldq % 4 == 0 && q_off % 4 == 0 && (dkv_off < 0 || (ld % 4 == 0 && dkv_off % 4 == 0)) &&
+      ((uintptr_t)qproj | (uintptr_t)proj | (uintptr_t)cw | (uintptr_t)pages | (uintptr_t)qn | (uintptr_t)qa) % 16 == 0) {
+    TLC_DISPATCH_DTYPE(dtype, TC, tlc_launch(latent_prepare_vec_kernel<TC>, dim3(T), dim3(nt), (size_t)rot * sizeof(float), stream, qproj, ldq,
+                                             q_off, proj, ld, dkv_off, cw, eps, inv_freq, rot, positions, row_seq, slots, block_table, max_pages,
+                                             (TC*)pages, (TC*)qn, (TC*)qa, H, dn, r, R, amplitude));
+    TLC_CHECK_LAUNCH("latent_prepare");
+    return 0;
+  }
   TLC_DISPATCH_DTYPE(dtype, TC, tlc_launch(latent_prepare_kernel<TC>, dim3(T), dim3(nt), 0, stream, qproj, ldq, q_off, proj, ld, dkv_off, cw, eps,
                                            inv_freq, rot, positions, row_seq, slots, block_table, max_pages, (TC*)pages, (TC*)qn,
                                            (TC*)qa, H, dn, r, R, amplitude));

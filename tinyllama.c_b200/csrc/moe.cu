@@ -4,8 +4,8 @@
 // the largest scores (the lowest index wins a tie); its weights are the chosen scores as they are.  The kernel also
 // sorts the (token, choice) pairs by expert -- counts, offsets, and for every expert the list of its pairs -- so that
 // each expert's rows form one contiguous range of a permutation; nothing goes through the host, so the same launches
-// serve any routing (and a captured graph).  tlc_moe_route_table needs no logits: a table gives every token id its experts,
-// all of one weight.
+// serve any routing (and a captured graph).  tlc_moe_route_tables needs no logits: a table gives every token id its
+// experts, all of one weight; it depends on the step's tokens alone, so one launch serves every layer of a model.
 //
 // Experts (tlc_moe_gate_up, tlc_moe_down): an expert is fed the token scaled by its weight, expert(w h); gate and up are
 // linear, so W (w h) = w (W h) and the epilogue of the first product applies w in 32 bits: act(w g) * (w u).  The
@@ -91,58 +91,80 @@ moe_topk_kernel(const float* __restrict__ logits, int ld, int T, int E, int top,
   }
 }
 
-// What the sort is told instead of ids where a table routes: a token's experts are the row of `table` [V, top] that its id
-// names, each with the same weight; the kernel then writes ids and weights itself.
-struct MoeTable {
-  const int* tokens;
-  const int* table;
-  int V, top;
-  float weight;
-  int* ids;
-  float* wts;
-};
-
-// One block sorts the pairs by expert: counts, offsets (and every expert's first tile of `tm` sorted rows), then the
-// list order [T*top]: pair index (t * top + k) of every sorted position.
-__global__ void __launch_bounds__(1024)
-moe_sort_kernel(const int* ids, int n_pairs, int E, int E_tiled, int tm, int* __restrict__ order,
-                int* __restrict__ offsets, int* __restrict__ tile_off, MoeTable by_table) {
-  tlc_pdl(ids, order, offsets, tile_off, by_table.ids, by_table.wts);
-  extern __shared__ int shi[];
+// A block sorts the pairs by expert: counts, offsets (and every expert's first tile of `tm` sorted rows), then the list order
+// [n_pairs]: pair index (t * top + k) of every sorted position.  shi: 2 * E ints.  ids[i] is read by the thread that owns i
+// (i modulo the block) only.
+__device__ __forceinline__ void moe_sort_pairs(const int* ids, int n_pairs, int E, int E_tiled, int tm, int* __restrict__ order,
+                                               int* __restrict__ offsets, int* __restrict__ tile_off, int* shi) {
   int* count = shi;            // [E]
   int* cursor = shi + E;       // [E]
   for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
   __syncthreads();
-  if (by_table.table) {
-    ids = by_table.ids;
-    for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
-      const int t = i / by_table.top;
-      int tok = by_table.tokens[t];
-      tok = tok < 0 ? 0 : (tok >= by_table.V ? by_table.V - 1 : tok);
-      int e = by_table.table[(size_t)tok * by_table.top + (i - t * by_table.top)];
-      e = e < 0 ? 0 : (e >= E ? E - 1 : e);             // (the host checks the table; never index out of bounds)
-      by_table.ids[i] = e;                              // (read again below by this thread only)
-      by_table.wts[i] = by_table.weight;
-      atomicAdd(&count[e], 1);
-    }
-  } else {
-    for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) atomicAdd(&count[ids[i]], 1);
-  }
+  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) atomicAdd(&count[ids[i]], 1);
   __syncthreads();
-  if (threadIdx.x == 0) {
-    int o = 0, tiles = 0;
-    for (int e = 0; e < E; e++) {
-      offsets[e] = o;
-      tile_off[e] = tiles;
-      cursor[e] = o;
-      o += count[e];
-      if (e < E_tiled) tiles += (count[e] + tm - 1) / tm;       // (the others have no weights: no product visits them)
+  if (threadIdx.x < 32) {      // running sums of pairs and tiles, 32 experts at a time
+    const int lane = threadIdx.x;
+    int pairs = 0, tiles = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + lane, c = e < E ? count[e] : 0;
+      const int k = e < E_tiled ? (c + tm - 1) / tm : 0;       // (the others have no weights: no product visits them)
+      int ci = c, ki = k;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int a = __shfl_up_sync(0xffffffffu, ci, o), b = __shfl_up_sync(0xffffffffu, ki, o);
+        if (lane >= o) { ci += a; ki += b; }
+      }
+      if (e < E) {
+        offsets[e] = cursor[e] = pairs + ci - c;
+        tile_off[e] = tiles + ki - k;
+      }
+      pairs += __shfl_sync(0xffffffffu, ci, 31);
+      tiles += __shfl_sync(0xffffffffu, ki, 31);
     }
-    offsets[E] = o;
-    tile_off[E] = tiles;
+    if (lane == 0) {
+      offsets[E] = pairs;
+      tile_off[E] = tiles;
+    }
   }
   __syncthreads();
   for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) order[atomicAdd(&cursor[ids[i]], 1)] = i;
+}
+
+__global__ void __launch_bounds__(1024)
+moe_sort_kernel(const int* __restrict__ ids, int n_pairs, int E, int E_tiled, int tm, int* __restrict__ order,
+                int* __restrict__ offsets, int* __restrict__ tile_off) {
+  tlc_pdl(ids, order, offsets, tile_off);
+  extern __shared__ int shi[];
+  moe_sort_pairs(ids, n_pairs, E, E_tiled, tm, order, offsets, tile_off, shi);
+}
+
+// Routing without a router, for all layers of a model that route this way: block p takes table p.  desc [n, 4] (64-bit): the
+// table's address (int [V, top]), its experts E, top, and whether its products may take tiles of 64 rows (they do when an
+// expert gets 64 rows or more on average).  Block p writes ids | order | offsets | tile_off from ints + p * ld_ints and the
+// weights, 1 / top each, from wts + p * ld_wts.
+__global__ void __launch_bounds__(1024)
+moe_route_tables_kernel(const int* __restrict__ tokens, const long long* __restrict__ desc, int T, int V, int* ints, int ld_ints, float* wts,
+                        int ld_wts) {
+  tlc_pdl(tokens, ints, wts);
+  extern __shared__ int shi[];
+  const long long* d = desc + 4 * (size_t)blockIdx.x;
+  const int* table = reinterpret_cast<const int*>(d[0]);
+  const int E = (int)d[1], top = (int)d[2], n_pairs = T * top;
+  const int tm = (d[3] && (long long)n_pairs >= 64LL * E) ? 64 : 32;
+  int* ids = ints + (size_t)blockIdx.x * ld_ints;
+  float* w = wts + (size_t)blockIdx.x * ld_wts;
+  const float weight = 1.0f / (float)top;
+  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
+    const int t = i / top;
+    int tok = tokens[t];
+    tok = tok < 0 ? 0 : (tok >= V ? V - 1 : tok);
+    const int e = table[(size_t)tok * top + (i - t * top)];
+    ids[i] = e < 0 ? 0 : (e >= E ? E - 1 : e);          // (tables are checked when they are bound; never index out of bounds)
+    w[i] = weight;
+  }
+  int* order = ids + n_pairs;
+  int* offsets = order + n_pairs;
+  moe_sort_pairs(ids, n_pairs, E, E, tm, order, offsets, offsets + E + 1, shi);
 }
 
 extern "C" int tlc_moe_route(const float* logits, int ld, int T, int E, int top, int mode, const float* choice_bias, int n_identity,
@@ -156,19 +178,18 @@ extern "C" int tlc_moe_route(const float* logits, int ld, int T, int E, int top,
   tlc_launch(moe_topk_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, logits, ld, T, E, top, mode, choice_bias, ids, wts, sum_to);
   TLC_CHECK_LAUNCH("moe_topk");
   tlc_launch(moe_sort_kernel, dim3(1), dim3(1024), (size_t)2 * E * sizeof(int), stream, (const int*)ids, T * top, E, E - n_identity, tile_rows,
-             order, offsets, tile_off, MoeTable{nullptr, nullptr, 0, 1, 0.f, nullptr, nullptr});
+             order, offsets, tile_off);
   TLC_CHECK_LAUNCH("moe_sort");
   return 0;
 }
 
-extern "C" int tlc_moe_route_table(const int* tokens, const int* table, int T, int V, int E, int top, float weight, int* ids, float* wts,
-                                   int* order, int* offsets, int* tile_off, int tile_rows, cudaStream_t stream) {
-  if (T == 0) return 0;
-  TLC_REQUIRE(tile_rows >= 1, "moe_route_table: tiles of %d rows", tile_rows);
-  TLC_REQUIRE(E >= 1 && top >= 1 && top <= E && E <= 4096 && V >= 1, "moe_route_table: %d experts, %d chosen, %d token ids", E, top, V);
-  tlc_launch(moe_sort_kernel, dim3(1), dim3(1024), (size_t)2 * E * sizeof(int), stream, (const int*)nullptr, T * top, E, E, tile_rows,
-             order, offsets, tile_off, MoeTable{tokens, table, V, top, weight, ids, wts});
-  TLC_CHECK_LAUNCH("moe_route_table");
+extern "C" int tlc_moe_route_tables(const int* tokens, const long long* desc, int n, int T, int V, int max_experts, int* ints, int ld_ints,
+                                    float* wts, int ld_wts, cudaStream_t stream) {
+  if (T == 0 || n == 0) return 0;
+  TLC_REQUIRE(max_experts >= 1 && max_experts <= 4096 && V >= 1, "moe_route_tables: %d experts, %d token ids", max_experts, V);
+  tlc_launch(moe_route_tables_kernel, dim3(n), dim3(1024), (size_t)2 * max_experts * sizeof(int), stream, tokens, desc, T, V, ints, ld_ints,
+             wts, ld_wts);
+  TLC_CHECK_LAUNCH("moe_route_tables");
   return 0;
 }
 

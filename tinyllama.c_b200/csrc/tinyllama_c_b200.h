@@ -126,10 +126,11 @@ int tlc_rmsnorm_shift(const float* x, const float* w, const float* mu, float eps
 /* res[t] (+)= y[t] / sqrt(mean(y[t]^2) + eps) * w (w NULL: y[t] itself) with y[t] = sum over p < n_parts of
  * parts[t, p, :] + g[t] * extra[t, :]; parts float [T, n_parts, D] (NULL with n_parts 0), extra float [T, D] or NULL,
  * g[t] = gate[t * gate_ld] (its sigmoid with gate_sigmoid; 1 with gate NULL), res float [T, D].  copy (or NULL): [T, D]
- * of type copy_dtype that receives the new res as well. */
+ * of type copy_dtype that receives the new res as well; with next_w [D] the RMS norm of the new res instead (eps next_eps,
+ * weight next_w): what the sublayer that follows reads. */
 int tlc_rmsnorm_add(const float* parts, int n_parts, const float* extra, const float* gate, int gate_ld,
                     int gate_sigmoid, const float* w, float eps, int T, int D, float* res, int accumulate,
-                    void* copy, int copy_dtype, cudaStream_t stream);
+                    void* copy, int copy_dtype, const float* next_w, float next_eps, cudaStream_t stream);
 
 /* ---- linear layers (gemm_tcgen05.cu, gemm_simt.cu) ----------------------------------------------------
  * out[m, n] (+)= (sum_k a[m, k] w[n, k]) * colscale[n] + colbias[n];  a [M, K], w [N, K], 32-bit sums.
@@ -341,6 +342,21 @@ int tlc_gate_mul(void* x, int dtype, int ldx, const float* gate, int ldg, int n,
 int tlc_qk_whole_norm(float* qkv, int ld, int q_off, int q_n, const float* qw, int k_off, int k_n, const float* kw, float eps,
                       int T, int q_count, int k_count, cudaStream_t stream);
 
+/* ---- from the projection of queries, keys and values to attention in one kernel (qkv_prepare.cu) -----------------
+ * On the C = (H + 2 KV) * hd columns (queries | keys | values) from `off` of the float projection proj [T, ld]: a causal
+ * convolution over time with K taps w [K, C] (K = 1, w NULL: none; state float [n_slots, K - 1, C]: every sequence's last
+ * projected rows), an RMS norm over all query columns and one over all key columns (q_w [H * hd], k_w [KV * hd], both or
+ * neither; q_count, k_count: how many columns hold values), a rotation of neighbouring pairs of every query and key head's
+ * first `rot` dimensions (cosines and sines times amplitude), then either out float [T, C], or q_out [T, H * hd] and the pages
+ * of keys and values, of `dtype`.  single_rows: every sequence brings one row; all_fresh: every sequence starts at
+ * position 0. */
+int tlc_qkv_prepare_ok(int H, int KV, int hd, int K, int ld, int off);
+int tlc_qkv_prepare(const float* proj, int ld, int off, const float* w, int K, float* state, const float* q_w, const float* k_w,
+                    int q_count, int k_count, float eps, const float* inv_freq, int rot, float amplitude, const int* positions,
+                    const int* row_seq, const int* cu_seqlens, const int* slots, const int* start_pos, const int* block_table,
+                    int max_pages, float* out, void* q_out, void* k_pages, void* v_pages, int dtype, int T, int B, int H, int KV,
+                    int hd, int single_rows, int all_fresh, cudaStream_t stream);
+
 /* ---- gated delta rule (delta_rule.cu) -------------------------------------------------------------------
  * Per head: M <- a M; w = b (v - M^T k); M <- M + k w^T; r = M^T q (a the decay, b the write strength `beta`), with M
  * [dk, dv] float per (slot, head) in state
@@ -371,9 +387,12 @@ int tlc_delta_rule(const float* qkv, int ld, int q_off, int k_off, int v_off, co
  * multiplied by sum_to. */
 int tlc_moe_route(const float* logits, int ld, int T, int E, int top, int mode, const float* choice_bias, int n_identity,
                   int* ids, float* wts, int* order, int* offsets, int* tile_off, int tile_rows, float sum_to, cudaStream_t stream);
-/* The same without a router: token t's experts are table[tokens[t], :] (int [V, top], distinct), each with weight `weight`. */
-int tlc_moe_route_table(const int* tokens, const int* table, int T, int V, int E, int top, float weight, int* ids, float* wts,
-                        int* order, int* offsets, int* tile_off, int tile_rows, cudaStream_t stream);
+/* The same without a router, for n tables at once: desc [n, 4] (64-bit, on the device) gives a table's address (int [V, top], the
+ * entries of a row distinct), its experts E (at most max_experts), top, and whether its products may take tiles of 64 rows (they
+ * do when T * top >= 64 E); token t's experts are the row tokens[t], each with weight 1 / top.  Table p's ids [T*top], order
+ * [T*top], offsets [E+1] and tile_off [E+1] follow one another from ints + p * ld_ints, its weights lie at wts + p * ld_wts. */
+int tlc_moe_route_tables(const int* tokens, const long long* desc, int n, int T, int V, int max_experts, int* ints, int ld_ints,
+                         float* wts, int ld_wts, cudaStream_t stream);
 /* y[pair, :D] = wts[pair] * x[token(pair), :D] for every pair with ids[pair] >= E. */
 int tlc_moe_identity(const void* x, int x_dtype, int ldx, const int* ids, const float* wts, int T, int top, int E, int D,
                      float* y, cudaStream_t stream);

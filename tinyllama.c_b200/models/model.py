@@ -16,6 +16,7 @@ from .. import ops
 from ..parts.base import (ChunkRequest, KVRequest, LayerCache, LayerRun, LayerSpec, Part, PartSpec, StateRequest, StepInfo, WeightSpec,
                           step_scratch)
 from ..parts.block import Block
+from ..parts.feed_forward import MoEFeedForward
 from ..parts.linear import StackedLinear, matrix_dtype
 
 
@@ -69,6 +70,7 @@ class Model:
         self.row_tables = {k: int(v) for k, v in (row_tables or {}).items()}
         self.rows_of: Dict[str, torch.Tensor] = {}
         self.embed_table: Optional[torch.Tensor] = None
+        self.by_table: List[MoEFeedForward] = []
         self.dtype: Optional[torch.dtype] = None
         self.device: Optional[torch.device] = None
 
@@ -112,6 +114,9 @@ class Model:
         for layer in self.layers:
             layer.bind(tensors, dtype, device)
         self.final_norm.bind(tensors, dtype, device)
+        self.by_table = [l.ffn for l in self.layers if isinstance(l.ffn, MoEFeedForward) and l.ffn.table is not None] \
+            if self.device.type == "cuda" else []
+        self.expert_tables = ops.ExpertTables([p.table_entry() for p in self.by_table]) if self.by_table else None
         self.rows_of = {name: tensors[name].to(device=device, dtype=torch.float32).contiguous() for name in self.row_tables}
         emb = tensors[self.embed_name]
         self.embed_table = emb.to(device=device, dtype=matrix_dtype(emb.dtype, dtype)).contiguous()
@@ -130,8 +135,10 @@ class Model:
         wait, what earlier steps left in the cache (never what a kernel of this step writes)."""
         x = torch.empty((step.n_rows, self.hidden), dtype=torch.float32, device=self.device)
         ops.embed(step.tokens, self.embed_table, self.embed_scale, x)
+        if self.by_table:                              # experts that token ids choose: all layers' routing at once
+            MoEFeedForward.route_step(self.by_table, self.expert_tables, step)
         with step_scratch(step):                       # the layers share the step's temporaries
-            ready = False                              # whether a layer left the stream in the activation type for the next
+            ready = False                              # whether a layer left the next one's input (Block.entry)
             for r, run in enumerate(self.schedule):
                 if run.add is not None:            # a learned row joins the stream before this entry (a pass of a repeated range)
                     ops.add_row(x, self.rows_of[run.add[0]][run.add[1]])
@@ -140,7 +147,7 @@ class Model:
                     ops.embed_add(step.tokens, self.embed_table, self.embed_scale, x)
                     ready = False
                 nxt = self.schedule[r + 1] if r + 1 < len(self.schedule) else None
-                wanted = nxt is not None and self.layers[nxt.layer].reads_stream_copy and nxt.add is None and not nxt.add_embedding
+                wanted = self.layers[nxt.layer].entry if nxt is not None and nxt.add is None and not nxt.add_embedding else None
                 ready = self.layers[run.layer].forward(x, step, cache.layer_view(r if run.cache is None else run.cache, run.writes,
                                                                                  run.kv_cache), ready, wanted)
         if want_rows is None or want_rows.numel() == 0:

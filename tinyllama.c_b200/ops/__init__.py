@@ -99,6 +99,9 @@ _SIGNATURES = {
     "tlc_convert": (_i, [_vp, _i, _i, _i, _vp, _i, _i, _i, _vp]),
     "tlc_softcap": (_i, [_vp, _ll, _f, _vp]),
     "tlc_rmsnorm_mean_add": (_i, [_vp, _i, _vp, _f, _f, _vp, _f, _i, _i, _vp, _i, _vp, _i, _vp]),
+    "tlc_qkv_prepare_ok": (_i, [_i, _i, _i, _i, _i, _i]),
+    "tlc_qkv_prepare": (_i, [_vp, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _f, _vp, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp,
+                             _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp]),
     "tlc_qk_whole_norm": (_i, [_vp, _i, _i, _i, _vp, _i, _i, _vp, _f, _i, _i, _i, _vp]),
     "tlc_shift_mix": (_i, [_vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp]),
     "tlc_wkv_scan": (_i, [_vp, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _vp]),
@@ -113,7 +116,7 @@ _SIGNATURES = {
                                    _i, _i, _vp, _i, _i, _vp]),
     "tlc_moe_identity": (_i, [_vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _vp, _vp]),
     "tlc_rmsnorm_shift": (_i, [_vp, _vp, _vp, _f, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp]),
-    "tlc_rmsnorm_add": (_i, [_vp, _i, _vp, _vp, _i, _i, _vp, _f, _i, _i, _vp, _i, _vp, _i, _vp]),
+    "tlc_rmsnorm_add": (_i, [_vp, _i, _vp, _vp, _i, _i, _vp, _f, _i, _i, _vp, _i, _vp, _i, _vp, _f, _vp]),
     "tlc_latent_prepare": (_i, [_vp, _i, _i, _vp, _i, _i, _vp, _f, _vp, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i,
                                 _i, _i, _f, _vp]),
     "tlc_latent_attention": (_i, [_vp, _vp, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _vp, _i, _vp]),
@@ -128,7 +131,7 @@ _SIGNATURES = {
     "tlc_moe_experts_mma": (_i, [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp, _i, _i, _i, _f, _f, _vp]),
     "tlc_mingru_scan": (_i, [_vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _vp, _vp]),
     "tlc_moe_route": (_i, [_vp, _i, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _f, _vp]),
-    "tlc_moe_route_table": (_i, [_vp, _vp, _i, _i, _i, _i, _f, _vp, _vp, _vp, _vp, _vp, _i, _vp]),
+    "tlc_moe_route_tables": (_i, [_vp, _vp, _i, _i, _i, _i, _vp, _i, _vp, _i, _vp]),
     "tlc_moe_gate_up": (_i, [_vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _i, _i, _i, _f, _f, _vp]),
     "tlc_qk_rotate_norm": (_i, [_vp, _i, _i, _i, _i, _i, _i, _i, _vp, _i, _i, _f, _vp, _i, _vp, _vp, _f, _f, _vp]),
     "tlc_gate_mul": (_i, [_vp, _i, _i, _vp, _i, _i, _i, _i, _vp]),
@@ -464,12 +467,13 @@ def rmsnorm_shift(x: torch.Tensor, weight: torch.Tensor, mix: torch.Tensor, eps:
 
 def rmsnorm_add(parts: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float, residual: torch.Tensor,
                 extra: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_sigmoid: bool = False,
-                accumulate: bool = True, copy: Optional[torch.Tensor] = None) -> None:
+                accumulate: bool = True, copy: Optional[torch.Tensor] = None, next_weight: Optional[torch.Tensor] = None,
+                next_eps: float = 0.0) -> None:
     """residual[t] (+)= rmsnorm(y[t]) * weight (weight None: y[t] itself) with y[t] = sum_p parts[t, p, :] + g[t] *
     extra[t, :]; parts float32 [T, D] or [T, n, D], extra float32 [T, D], gate float32 [T] or one column of a wider
     float32 matrix; g is the gate, or its sigmoid.  copy [T, D] (float32 or bfloat16, contiguous) receives the new
-    residual rows as well."""
-    _gpu(parts, weight, residual, extra, gate, copy)
+    residual rows as well; with next_weight (float32 [D]) their RMS norm with that weight and next_eps instead."""
+    _gpu(parts, weight, residual, extra, gate, copy, next_weight)
     T, D = residual.shape
     n = 0
     if parts is not None:
@@ -486,8 +490,10 @@ def rmsnorm_add(parts: Optional[torch.Tensor], weight: Optional[torch.Tensor], e
     if residual.dtype != torch.float32 or not residual.is_contiguous():
         raise KernelError("rmsnorm_add: the residual stream must be contiguous float32")
     _f32vec(weight, D, "rmsnorm_add weight")
+    _f32vec(next_weight, D, "rmsnorm_add next norm's weight")
     _call("tlc_rmsnorm_add", _p(parts), n, _p(extra), _p(gate), int(gate_ld), int(bool(gate_sigmoid)), _p(weight), float(eps),
-          T, D, residual.data_ptr(), int(bool(accumulate)), *_copy_of(copy, T, D, "rmsnorm_add"), _stream())
+          T, D, residual.data_ptr(), int(bool(accumulate)), *_copy_of(copy, T, D, "rmsnorm_add"), _p(next_weight), float(next_eps),
+          _stream())
 
 
 def _copy_of(copy: Optional[torch.Tensor], T: int, D: int, what: str):
@@ -1153,6 +1159,13 @@ def _moe_mma_ok(x: torch.Tensor, w_gate_up: torch.Tensor, act_dtype: torch.dtype
                                                  0, w_gate_up.data_ptr(), D))
 
 
+def moe_tiles_of_64(w_gate_up: torch.Tensor, run_dtype: torch.dtype, F: int) -> bool:
+    """Whether dense rows of the run's type may take tiles of 64 rows in the experts' products (see moe_tile_rows)."""
+    D = w_gate_up.shape[2]
+    return bool(run_dtype == torch.bfloat16 and F % 8 == 0 and D % 8 == 0
+                and library().tlc_grouped_mma_ok(BF16, dtype_code(w_gate_up.dtype), None, D, 0, w_gate_up.data_ptr(), D))
+
+
 def moe_tile_rows(x: torch.Tensor, w_gate_up: torch.Tensor, act_dtype: torch.dtype, top: int, F: Optional[int] = None) -> int:
     """Rows of a tile of the experts' products for this input: 64 where the tensor-core kernel runs and an expert gets
     64 rows or more on average, else 32.  The routing is made for that number (moe_route) and carries it."""
@@ -1197,21 +1210,44 @@ def moe_route(logits: torch.Tensor, n_experts: int, top: int, tile_rows: int = 3
     return ids, wts, order, offsets, tile_off, int(tile_rows)
 
 
-def moe_route_table(tokens: torch.Tensor, table: torch.Tensor, n_experts: int, weight: float, tile_rows: int = 32):
-    """Routing without a router: row t's experts are table[tokens[t]] (int32 [V, top], the entries of a row distinct and below
-    n_experts), every one of them with the same weight.  Returns what moe_route does."""
-    _gpu(tokens, table)
+class ExpertTables:
+    """Tables that give every token id its experts (int32 [V, top], the entries of a row distinct), of one or several layers:
+    what moe_route_tables() routes by in one launch.  tables: (table on the device, number of experts, whether the experts'
+    products may take tiles of 64 rows) each."""
+
+    def __init__(self, tables):
+        self.tables = [t for t, _, _ in tables]
+        self.sizes = [(int(E), int(t.shape[1]), bool(tiles_64)) for t, E, tiles_64 in tables]
+        self.vocab = int(self.tables[0].shape[0])
+        for t in self.tables:
+            _i32(t, "expert table")
+            if t.dim() != 2 or t.shape[0] != self.vocab:
+                raise KernelError("expert tables: int32 [V, top] of one vocabulary")
+        self.max_experts = max(E for E, _, _ in self.sizes)
+        self.desc = torch.tensor([[t.data_ptr(), E, top, int(k)] for t, (E, top, k) in zip(self.tables, self.sizes)], dtype=torch.int64,
+                                 device=self.tables[0].device)
+        self.desc_32 = self.desc.clone()             # the same with tiles of 32 rows only (see grouped_mma)
+        self.desc_32[:, 3] = 0
+
+
+def moe_route_tables(tokens: torch.Tensor, tables: ExpertTables) -> list:
+    """Routing without a router: row t's experts in every table are its row tokens[t], each weighted 1 / top.  Returns, table by
+    table, what moe_route does."""
+    _gpu(tokens, tables.desc)
     _i32(tokens, "tokens")
-    _i32(table, "expert table")
-    T, (V, top) = tokens.numel(), table.shape
-    ints = torch.empty(2 * T * top + 2 * (n_experts + 1), dtype=torch.int32, device=tokens.device)
-    ids, order = ints[:T * top], ints[T * top:2 * T * top]
-    offsets = ints[2 * T * top:2 * T * top + n_experts + 1]
-    tile_off = ints[2 * T * top + n_experts + 1:]
-    wts = torch.empty(T * top, dtype=torch.float32, device=tokens.device)
-    _call("tlc_moe_route_table", tokens.data_ptr(), table.data_ptr(), T, V, int(n_experts), top, float(weight), ids.data_ptr(),
-          wts.data_ptr(), order.data_ptr(), offsets.data_ptr(), tile_off.data_ptr(), int(tile_rows), _stream())
-    return ids, wts, order, offsets, tile_off, int(tile_rows)
+    T = tokens.numel()
+    ld_ints, ld_wts = max(2 * T * top + 2 * (E + 1) for E, top, _ in tables.sizes), max(T * top for _, top, _ in tables.sizes)
+    ints = torch.empty((len(tables.sizes), ld_ints), dtype=torch.int32, device=tokens.device)
+    wts = torch.empty((len(tables.sizes), ld_wts), dtype=torch.float32, device=tokens.device)
+    desc = tables.desc if _grouped_mma else tables.desc_32
+    _call("tlc_moe_route_tables", tokens.data_ptr(), desc.data_ptr(), len(tables.sizes), T, tables.vocab, tables.max_experts,
+          ints.data_ptr(), ld_ints, wts.data_ptr(), ld_wts, _stream())
+    out = []
+    for p, (E, top, tiles_64) in enumerate(tables.sizes):
+        n, row = T * top, ints[p]
+        out.append((row[:n], wts[p, :n], row[n:2 * n], row[2 * n:2 * n + E + 1], row[2 * n + E + 1:2 * n + 2 * (E + 1)],
+                    64 if tiles_64 and _grouped_mma and n >= 64 * E else 32))
+    return out
 
 
 def moe_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, routing, top: int, act: torch.Tensor,
@@ -1274,6 +1310,57 @@ def qk_whole_norm(qkv: torch.Tensor, q_off: int, q_n: int, q_weight: torch.Tenso
     _f32vec(k_weight, k_n, "key norm weight")
     _call("tlc_qk_whole_norm", qkv.data_ptr(), ld, int(q_off), int(q_n), q_weight.data_ptr(), int(k_off), int(k_n),
           k_weight.data_ptr(), float(eps), qkv.shape[0], int(q_count or q_n), int(k_count or k_n), _stream())
+
+
+DISABLE_QKV_PREPARE = bool(int(os.environ.get("TLC_DISABLE_QKV_PREPARE", "0")))
+
+
+def qkv_prepare_ok(H: int, KV: int, hd: int, taps: int, ld: int, off: int) -> bool:
+    """Whether qkv_prepare takes these sizes (else the convolution, the norm, the rotation and the stores are kernels of their
+    own; TLC_DISABLE_QKV_PREPARE=1 keeps them that way)."""
+    return not DISABLE_QKV_PREPARE and bool(library().tlc_qkv_prepare_ok(int(H), int(KV), int(hd), int(taps), int(ld), int(off)))
+
+
+def qkv_prepare(proj: torch.Tensor, off: int, H: int, KV: int, hd: int, inv_freq: torch.Tensor, amplitude: float, step,
+                taps: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None, q_weight: Optional[torch.Tensor] = None,
+                k_weight: Optional[torch.Tensor] = None, eps: float = 0.0, q_count: Optional[int] = None, k_count: Optional[int] = None,
+                out: Optional[torch.Tensor] = None, q_out: Optional[torch.Tensor] = None, k_pages: Optional[torch.Tensor] = None,
+                v_pages: Optional[torch.Tensor] = None, block_table: Optional[torch.Tensor] = None) -> None:
+    """In one kernel, on the columns queries | keys | values from `off` of the float32 projection proj [T, *] (H, KV and KV
+    heads of hd): the convolution over time (taps float32 [K, C], state as in channel_conv; None: none), the norms over all
+    query and all key columns (weights float32, both or neither; q_count, k_count as in qk_whole_norm), the rotation of
+    neighbouring pairs by position * inv_freq[i] with cosines and sines times amplitude, and then out float32 [T, C], or (out
+    None) q_out [T, H*hd] and the sequences' pages."""
+    _gpu(proj, inv_freq, taps, state, q_weight, k_weight, out, q_out, k_pages, v_pages, block_table)
+    T, C = proj.shape[0], (H + 2 * KV) * hd
+    K = 1 if taps is None else taps.shape[0]
+    ld = _rows(proj, "qkv_prepare input")
+    if proj.dtype != torch.float32 or off + C > max(ld, proj.shape[1]):
+        raise KernelError("qkv_prepare: a float32 projection that holds queries, keys and values")
+    if taps is not None:
+        _f32vec(taps, K * C, "qkv_prepare taps")
+    _f32vec(q_weight, H * hd, "query norm weight")
+    _f32vec(k_weight, KV * hd, "key norm weight")
+    _f32vec(inv_freq, inv_freq.numel(), "rotation inv_freq")
+    dtype = F32
+    if out is not None:
+        if out.dtype != torch.float32 or not out.is_contiguous() or tuple(out.shape) != (T, C):
+            raise KernelError("qkv_prepare: out must be contiguous float32 [T, C]")
+    else:
+        _i32(block_table, "block_table")
+        dtype = dtype_code(q_out.dtype)
+        if k_pages.dtype != q_out.dtype or v_pages.dtype != q_out.dtype or not q_out.is_contiguous() or tuple(q_out.shape) != (T, H * hd) \
+                or not k_pages.is_contiguous() or not v_pages.is_contiguous() or tuple(k_pages.shape[1:]) != (KV, PAGE, hd):
+            raise KernelError("qkv_prepare: q_out [T, H*hd] and pages [n, KV, 64, hd] contiguous and of one type")
+    global _launches
+    fresh, single = _all_fresh(step), int(step.max_new == 1)
+    if K > 1 and not fresh and not (single and T == step.n_seqs):
+        _launches += 1                  # (the kept rows are written by a kernel of their own)
+    _call("tlc_qkv_prepare", proj.data_ptr(), ld, int(off), _p(taps), K, _window(state, K, C, "qkv_prepare"), _p(q_weight), _p(k_weight),
+          int(q_count or H * hd), int(k_count or KV * hd), float(eps), inv_freq.data_ptr(), 2 * inv_freq.numel(), float(amplitude),
+          step.positions.data_ptr(), step.row_seq.data_ptr(), step.cu_seqlens.data_ptr(), step.slots.data_ptr(), step.start_pos.data_ptr(),
+          _p(block_table), 0 if block_table is None else block_table.shape[1], _p(out), _p(q_out), _p(k_pages), _p(v_pages), dtype, T,
+          step.n_seqs, H, KV, hd, single, fresh, _stream())
 
 
 # ---- time mixing with a decaying matrix state -------------------------------------------------------------------

@@ -17,7 +17,7 @@ Position      rotation_table() -> inverse frequencies (the kernels rotate q and 
               the 32-bit projection in place; storing keys and values is the mixer's business
 Mixer         forward(normed [T, D], step, cache, residual [T, D] float32)  adds its output into residual
 FeedForward   forward(normed [T, D], residual [T, D] float32)               adds its output into residual (one that says
-              takes_tokens = True is also given the rows' token ids, tokens=)
+              takes_step = True is also given the StepInfo, step=)
 All of them   weight_specs() -> [WeightSpec], bind(tensors, dtype, device)
 Mixers also   cache_requests() -> [KVRequest | StateRequest], step_requests() -> [ChunkRequest]
 """
@@ -299,3 +299,48 @@ def scratch_buf(tag: str, shape, dtype: torch.dtype, device) -> torch.Tensor:
     if t is None:
         t = _scratch[key] = torch.empty(shape, dtype=dtype, device=device)
     return t
+
+
+# ---- streams ---------------------------------------------------------------------------------------
+_streams = {}
+
+
+def current_stream(device) -> "torch.cuda.Stream":
+    """The current stream of the device as a torch object.  torch.cuda.current_stream() takes some 10 us of Python
+    a call and a block asks once a layer, so the object is kept by the stream's handle (which torch's raw query
+    gives in a fraction of that) and made anew only when the handle is a new one."""
+    index = device.index if device.index is not None else torch.cuda.current_device()
+    raw = getattr(torch._C, "_cuda_getCurrentRawStream", None)
+    if raw is None:
+        return torch.cuda.current_stream(index)
+    handle = raw(index)
+    hit = _streams.get((index, handle))
+    if hit is None:
+        if len(_streams) > 64:
+            _streams.clear()
+        hit = _streams[(index, handle)] = torch.cuda.current_stream(index)
+    return hit
+
+
+class SideStream:
+    """A stream of its own for work that runs beside what its caller launches next: run(f) starts after everything launched on
+    the current stream so far, join() makes the current stream wait for it.  (Under stream capture: a branch of the graph.)"""
+
+    def __init__(self, device):
+        self.device = torch.device(device)
+        self.stream = torch.cuda.Stream(device=self.device)
+        self.fork, self.done = torch.cuda.Event(), torch.cuda.Event()     # every wait follows its record in program order
+
+    def run(self, f: Callable[[], None]) -> None:
+        main = current_stream(self.device)
+        self.fork.record(main)
+        self.stream.wait_event(self.fork)
+        torch.cuda.set_stream(self.stream)        # (the context manager asks for the current stream again: 10 us)
+        try:
+            f()
+            self.done.record(self.stream)
+        finally:
+            torch.cuda.set_stream(main)
+
+    def join(self) -> None:
+        current_stream(self.device).wait_event(self.done)

@@ -15,8 +15,9 @@ from typing import Dict, List, Optional
 
 import torch
 
-from .base import LayerCache, LayerSpec, Part, StepInfo, WeightSpec, act_empty, scratch_buf, scratch_is_shared
+from .base import LayerCache, LayerSpec, Part, StepInfo, WeightSpec, current_stream, scratch_buf, scratch_is_shared
 from .linear import StackedLinear
+from .norm import RMSNorm
 
 
 # Mixers that are independent of one another between their input and output projections run side by side on
@@ -46,26 +47,6 @@ PROMPT_SIDE_BLOCKS = int(os.environ.get("TLC_PROMPT_SIDE_BLOCKS", "0"))
 # one after the other unless TLC_PARALLEL_FFN_PROMPTS=1.
 PARALLEL_FFN = int(os.environ.get("TLC_PARALLEL_FFN", "1"))
 PARALLEL_FFN_PROMPTS = bool(int(os.environ.get("TLC_PARALLEL_FFN_PROMPTS", "0")))
-
-
-_streams = {}
-
-
-def _current_stream(device) -> "torch.cuda.Stream":
-    """The current stream of the device as a torch object.  torch.cuda.current_stream() takes some 10 us of Python
-    a call and a block asks once a layer, so the object is kept by the stream's handle (which torch's raw query
-    gives in a fraction of that) and made anew only when the handle is a new one."""
-    index = device.index if device.index is not None else torch.cuda.current_device()
-    raw = getattr(torch._C, "_cuda_getCurrentRawStream", None)
-    if raw is None:
-        return torch.cuda.current_stream(index)
-    handle = raw(index)
-    hit = _streams.get((index, handle))
-    if hit is None:
-        if len(_streams) > 64:
-            _streams.clear()
-        hit = _streams[(index, handle)] = torch.cuda.current_stream(index)
-    return hit
 
 
 class Block(Part):
@@ -145,7 +126,7 @@ class Block(Part):
         other on the current stream, in the mixers' order, each after its mixer has finished.  (Under stream capture the
         side streams become parallel branches of the graph.)  outs [T, n, D]: every mixer's output projection is written
         to its own rows outs[:, i] instead (a layer that joins its mixers' results by something else than their sum)."""
-        main = _current_stream(x32.device)
+        main = current_stream(x32.device)
         if not hasattr(self, "_side"):
             self._side = [torch.cuda.Stream(device=x32.device) for _ in self.mixers[1:]]
             # events are made once: a record overwrites the event's last state, and every wait of this block follows
@@ -238,15 +219,15 @@ class Block(Part):
                 self._pre_norm(self.ffn_norm, x32, "block.ffn_normed", step, cache))
 
     def _ffn_more(self, step: StepInfo) -> dict:
-        """What the feed-forward is given beside its input: the rows' token ids, where it asks for them."""
-        return {"tokens": step.tokens} if getattr(self.ffn, "takes_tokens", False) else {}
+        """What the feed-forward is given beside its input: the step, where it asks for it."""
+        return {"step": step} if getattr(self.ffn, "takes_step", False) else {}
 
     def _two_branches(self, normed: torch.Tensor, x32: torch.Tensor, run_mixers, ffn_in: Optional[torch.Tensor], more: dict) -> None:
         """A parallel layer on two streams (under stream capture: two branches of the graph): the mixers, which add
         their outputs into the residual stream, and the feed-forward's terms; the terms are added after the branches have
         met, on the current stream, so the order of the sums is fixed.  run_mixers(): launches the mixers on whatever
         stream is current."""
-        main = _current_stream(x32.device)
+        main = current_stream(x32.device)
         if not hasattr(self, "_ffn_side"):
             least, greatest = torch.cuda.Stream.priority_range() if hasattr(torch.cuda.Stream, "priority_range") else (0, -1)
             self._ffn_side = torch.cuda.Stream(device=x32.device, priority=greatest if PARALLEL_FFN == 1 else least)
@@ -271,7 +252,7 @@ class Block(Part):
         main.wait_event(self._ffn_done)
         self.ffn.add_parts(terms, x32)
 
-    def _joined_mixers(self, x32: torch.Tensor, step: StepInfo, cache: LayerCache, copy: Optional[torch.Tensor] = None) -> None:
+    def _joined_mixers(self, x32: torch.Tensor, step: StepInfo, cache: LayerCache, next_entry=None) -> dict:
         """x <- x + out_norm(join(mixer_i(h))): every mixer's result in rows of its own, then the join (and the norm after
         it) in one kernel.  Mixers that offer their projections share the input product and, in one-token steps, run side
         by side on streams."""
@@ -293,27 +274,46 @@ class Block(Part):
                 if not self._mixer_overwrites[i]:
                     raise ValueError("a layer that joins its mixers' results needs mixers whose forward() can overwrite its target")
                 m.forward(x32 if reads[i] else normed, step, cache, outs[:, i], accumulate=False)
-        self.mixer_join.add_joined(outs, x32, self.mixer_out_norm, copy=copy)
+        left = self._leave_after_mixers(x32, next_entry) if self.mixer_out_norm is not None else {}
+        self.mixer_join.add_joined(outs, x32, self.mixer_out_norm, **left)
+        return left
 
-    # A sublayer without a norm in front reads the residual stream in the activation type.  The kernel that last added
-    # into the stream (an output norm) writes that copy as its second output, so that no kernel of its own has to make it:
-    # _stream_copy() names the buffer to the adding kernel and notes that it is filled, _pre_norm() then hands it over.
+    # What a sublayer reads is the residual stream in the activation type, or (behind a plain RMS norm) its norm.  The kernel
+    # that last added into the stream (an output norm) has the new rows in its hands and writes that as its second output, so
+    # that no kernel of its own has to make it: _leave() names the buffer to the adding kernel and notes that it is filled,
+    # _pre_norm() then hands it over.
     @property
-    def reads_stream_copy(self) -> bool:
-        """Whether this layer's first step is a copy of the residual stream in the activation type (no norm before the
-        mixers, and a mixer that does not take the 32-bit rows themselves)."""
-        return bool(self.mixers) and self._plain_copy(self.mixer_norm) \
-            and not all(bool(getattr(m, "reads_stream", False)) for m in self.mixers)
+    def entry(self):
+        """The norm in front of this layer's mixers, if the layer before may leave its result: none at all (a copy of the
+        stream in the activation type, unless the mixers take the 32-bit rows themselves), or a plain RMS norm."""
+        if not self.mixers or not (self._plain_copy(self.mixer_norm) or type(self.mixer_norm) is RMSNorm):
+            return None
+        if self._plain_copy(self.mixer_norm) and all(bool(getattr(m, "reads_stream", False)) for m in self.mixers):
+            return None
+        return self.mixer_norm
 
     @staticmethod
     def _plain_copy(norm) -> bool:
         return norm is not None and getattr(norm, "identity", False) and not hasattr(norm, "forward_step")
 
-    def _stream_copy(self, tag: str, x32: torch.Tensor) -> Optional[torch.Tensor]:
-        if not (x32.is_cuda and scratch_is_shared()):
-            return None
+    def _leave(self, norm, x32: torch.Tensor, tag: str, adds=None) -> dict:
+        """What the adding kernel of `adds` (an output norm; None: of a join, which leaves plain copies only) is told so that
+        it leaves `norm` of the new stream in buffer `tag`; nothing where it cannot."""
+        normed = type(norm) is RMSNorm and type(adds) is RMSNorm
+        if not (x32.is_cuda and scratch_is_shared()) or not (self._plain_copy(norm) or normed):
+            return {}
         self._copied.add(tag)
-        return scratch_buf(tag, x32.shape, self.dtype, x32.device)
+        out = {"copy": scratch_buf(tag, x32.shape, self.dtype, x32.device)}
+        if normed:
+            out["next_norm"] = norm
+        return out
+
+    def _leave_after_mixers(self, x32: torch.Tensor, next_entry, adds=None) -> dict:
+        """_leave() for the kernel that adds the mixers' result: the feed-forward's input, or in a layer without one the next
+        layer's (next_entry)."""
+        if self.ffn is None:
+            return self._leave(next_entry, x32, "block.normed", adds)
+        return {} if self.parallel_ffn else self._leave(self.ffn_norm, x32, "block.ffn_normed", adds)
 
     def _pre_norm(self, norm, x32: torch.Tensor, tag: str, step: StepInfo, cache: LayerCache) -> torch.Tensor:
         normed = scratch_buf(tag, x32.shape, self.dtype, x32.device)
@@ -326,21 +326,14 @@ class Block(Part):
             norm.forward(x32, normed)
         return normed
 
-    def forward(self, x32: torch.Tensor, step: StepInfo, cache: LayerCache, copy_ready: bool = False,
-                copy_for_next: bool = False) -> bool:
-        """Updates the float32 residual stream x32 [T, D] in place.  copy_ready: the layer before has left the stream in
-        the activation type where this layer's mixers look for it; copy_for_next: the next layer wants the same of this
-        one.  Returns whether that copy was written."""
-        self._copied = {"block.normed"} if copy_ready and self.reads_stream_copy and scratch_is_shared() else set()
-        last_add_is_mixers = self.ffn is None or self.parallel_ffn
-        copy = None
-        if self.mixers and self.mixer_out_norm is not None:
-            if last_add_is_mixers:
-                copy = self._stream_copy("block.normed", x32) if copy_for_next and self.ffn is None else None
-            elif self._plain_copy(self.ffn_norm):
-                copy = self._stream_copy("block.ffn_normed", x32)
+    def forward(self, x32: torch.Tensor, step: StepInfo, cache: LayerCache, entry_ready: bool = False, next_entry=None) -> bool:
+        """Updates the float32 residual stream x32 [T, D] in place.  entry_ready: the layer before has left what this layer's
+        `entry` makes of the stream where its mixers look for it; next_entry: the next layer's (None: not wanted).  Returns
+        whether this layer has left that for it."""
+        self._copied = {"block.normed"} if entry_ready and self.entry is not None and scratch_is_shared() else set()
+        left = {}
         if self.mixers and self.mixer_join is not None:
-            self._joined_mixers(x32, step, cache, copy)
+            left = self._joined_mixers(x32, step, cache, next_entry)
         elif self.mixers and self.mixer_out_norm is not None:
             # x <- x + out_norm(sum of the mixers' outputs); a mixer that reads the stream itself gets the 32-bit rows
             reads = [bool(getattr(m, "reads_stream", False)) and getattr(self.mixer_norm, "identity", False) for m in self.mixers]
@@ -353,7 +346,8 @@ class Block(Part):
                     m.forward(x32 if reads[i] else normed, step, cache, y, accumulate=i > 0)
                 else:
                     m.forward(x32 if reads[i] else normed, step, cache, y)
-            self.mixer_out_norm.add_normed(y, x32, copy=copy)
+            left = self._leave_after_mixers(x32, next_entry, self.mixer_out_norm)
+            self.mixer_out_norm.add_normed(y, x32, **left)
         elif self.mixers:
             normed, ffn_in = self._parallel_inputs(x32, step, cache) if self.parallel_ffn \
                 else (self._pre_norm(self.mixer_norm, x32, "block.normed", step, cache), None)
@@ -366,8 +360,8 @@ class Block(Part):
             self.ffn.forward(ffn_in, x32, **self._ffn_more(step))
             return False
         if self.ffn is not None:
-            return self._feed_forward(x32, step, cache, copy_for_next)
-        return copy is not None
+            return self._feed_forward(x32, step, cache, next_entry)
+        return bool(left)
 
     def _run_mixers(self, normed: torch.Tensor, x32: torch.Tensor, step: StepInfo, cache: LayerCache) -> None:
         """The mixers of a layer without a mixer output norm, from their shared normed input into the residual stream."""
@@ -389,12 +383,11 @@ class Block(Part):
             for m in self.mixers:
                 m.forward(normed, step, cache, x32)
 
-    def _feed_forward(self, x32: torch.Tensor, step: StepInfo, cache: LayerCache, copy_for_next: bool = False) -> bool:
+    def _feed_forward(self, x32: torch.Tensor, step: StepInfo, cache: LayerCache, next_entry=None) -> bool:
         """A feed-forward with a norm of its own, after the mixers.  Returns whether the kernel that added its result
-        also left the stream in the activation type for the next layer (copy_for_next)."""
+        also left the next layer's input (next_entry)."""
         normed = self._pre_norm(self.ffn_norm, x32, "block.ffn_normed", step, cache)
-        copy = self._stream_copy("block.normed", x32) if copy_for_next and self.ffn_out_norm is not None else None
-        self._copied.discard("block.normed")          # (the next layer is told by the return value)
+        left = self._leave(next_entry, x32, "block.normed", self.ffn_out_norm) if self.ffn_out_norm is not None else {}
         # without a norm in front, a feed-forward that can use them (takes_stream) also gets the 32-bit rows themselves
         more = self._ffn_more(step)
         if getattr(self.ffn_norm, "identity", False) and getattr(self.ffn, "takes_stream", False):
@@ -404,7 +397,7 @@ class Block(Part):
         elif hasattr(self.ffn, "forward_parts"):
             # a feed-forward whose result is a sum of terms hands them to the norm, which adds them up itself
             parts, extra, gate = self.ffn.forward_parts(normed, **more)
-            self.ffn_out_norm.add_normed(parts, x32, extra, gate, copy=copy)
+            self.ffn_out_norm.add_normed(parts, x32, extra, gate, **left)
         else:
             y = scratch_buf("block.ffn_out", x32.shape, torch.float32, x32.device)
             if self._ffn_overwrites:
@@ -412,5 +405,5 @@ class Block(Part):
             else:
                 y.zero_()
                 self.ffn.forward(normed, y, **more)
-            self.ffn_out_norm.add_normed(y, x32, copy=copy)
-        return copy is not None
+            self.ffn_out_norm.add_normed(y, x32, **left)
+        return bool(left)

@@ -8,13 +8,18 @@ the reference.
 """
 from __future__ import annotations
 
+import os
 from typing import Dict, List, Optional
 
 import torch
 
 from .. import ops
-from .base import Part, PartSpec, WeightSpec, act_empty, register_feed_forward, scratch_buf
+from .base import Part, PartSpec, SideStream, WeightSpec, register_feed_forward, scratch_buf
 from .linear import StackedLinear
+
+# In steps of at most this many rows a shared expert runs on a stream of its own beside the routed ones: its two products are
+# short kernels that would otherwise stand in the chain.  0: never.
+SHARED_BESIDE_ROWS = int(os.environ.get("TLC_SHARED_BESIDE_ROWS", "128"))
 
 
 @register_feed_forward("swiglu")
@@ -167,7 +172,7 @@ class MoEFeedForward(Part):
         """expert_names: patterns of gate, up, down with {e} for the expert's index.  weights_sum_to > 0 (weights
         "softmax_all"): a token's weights are the chosen scores divided by their sum (+ 1e-20) times this number.
         table_name: the tensor [vocab, top] that routes by token id (router_name is then None)."""
-        self.table_name, self.vocab, self.takes_tokens = table_name, int(vocab), table_name is not None
+        self.table_name, self.vocab, self.takes_step = table_name, int(vocab), table_name is not None
         if (table_name is None) == (router_name is None):
             raise ValueError("moe: a router or a table chooses the experts")
         if table_name is not None and (self.vocab < 1 or router_bias_name or choice_bias_name or n_identity or shared_gate_name
@@ -199,6 +204,7 @@ class MoEFeedForward(Part):
         if self.shared is None and shared_gate_name is not None:
             raise ValueError("moe: a shared expert's gate needs a shared expert")
         self.dtype = None
+        self._side = None
 
     def weight_specs(self) -> List[WeightSpec]:
         specs = [WeightSpec(self.router_name, (self.n_out, self.hidden))] if self.router_name else \
@@ -233,6 +239,7 @@ class MoEFeedForward(Part):
             if table.numel() and (int(table.min()) < 0 or int(table.max()) >= self.E):
                 raise ValueError(f"moe: '{self.table_name}' names experts outside 0..{self.E - 1}")
             self.table = table.to(device=device, dtype=torch.int32).contiguous()
+            self.expert_tables = None            # (made when this part routes by itself)
         self.router_bias = None
         if self.router_bias_name:                # added to the 32-bit logits in the product's epilogue (nothing on the shared gate's)
             self.router_bias = torch.zeros(self.router.shape[0], dtype=torch.float32, device=device)
@@ -256,24 +263,48 @@ class MoEFeedForward(Part):
 
     takes_stream = True        # forward(..., stream=x32): an expert that returns its input returns the 32-bit rows
 
-    def _route(self, normed: torch.Tensor, tokens: Optional[torch.Tensor]):
+    def table_entry(self):
+        """This part's table as ops.ExpertTables takes it."""
+        return self.table, self.E, ops.moe_tiles_of_64(self.w_gate_up, self.dtype, self.F)
+
+    @staticmethod
+    def route_step(parts, tables, step) -> None:
+        """Routes the step's rows for all of `parts` (which route by tables; tables: ops.ExpertTables of theirs) in one launch,
+        ahead of the layers: the routing depends on the tokens alone.  The parts find it in the step."""
+        for part, routing in zip(parts, ops.moe_route_tables(step.tokens, tables)):
+            step.scratch[("moe.routing", id(part))] = routing
+
+    def _route(self, normed: torch.Tensor, step):
         """(routing as moe_experts takes it, the router's logits or None)."""
-        tile_rows = ops.moe_tile_rows(normed, self.w_gate_up, self.dtype, self.top, self.F)
         if self.table is not None:
-            if tokens is None:
-                raise ValueError("moe: experts chosen by a table need the rows' token ids")
-            return ops.moe_route_table(tokens, self.table, self.E, 1.0 / self.top, tile_rows), None
+            if step is None:
+                raise ValueError("moe: experts chosen by a table need the step, for its token ids")
+            routing = step.scratch.get(("moe.routing", id(self)))
+            if routing is None:
+                if self.expert_tables is None:
+                    self.expert_tables = ops.ExpertTables([self.table_entry()])
+                routing = ops.moe_route_tables(step.tokens, self.expert_tables)[0]
+            return routing, None
+        tile_rows = ops.moe_tile_rows(normed, self.w_gate_up, self.dtype, self.top, self.F)
         logits = scratch_buf("moe.logits", (normed.shape[0], self.router.shape[0]), torch.float32, normed.device)
         ops.linear(normed, self.router, logits, None, self.router_bias)
         return ops.moe_route(logits, self.n_out, self.top, tile_rows, self.weights, self.choice_bias, self.n_identity,
                              self.weights_sum_to), logits
 
-    def forward_parts(self, normed: torch.Tensor, stream: Optional[torch.Tensor] = None, tokens: Optional[torch.Tensor] = None):
+    def forward_parts(self, normed: torch.Tensor, stream: Optional[torch.Tensor] = None, step=None):
         """(parts float32 [T, top, D], shared expert's output float32 [T, D] or None, its gate's logit float32 [T] or
         None): the result is sum_k parts[:, k] + sigmoid(logit) * shared (without a gate: + shared).  stream: the 32-bit rows that `normed` is a
         copy of, where the layer has no norm in front of this part (identity experts then return those)."""
         T, dev = normed.shape[0], normed.device
-        routing, logits = self._route(normed, tokens)
+        routing, logits = self._route(normed, step)
+        side = None
+        if self.shared is not None:
+            shared_out = scratch_buf("moe.shared", (T, self.hidden), torch.float32, dev)
+            if SHARED_BESIDE_ROWS and T <= SHARED_BESIDE_ROWS and normed.is_cuda:
+                if self._side is None:
+                    self._side = SideStream(dev)
+                side = self._side
+                side.run(lambda: self.shared.forward(normed, shared_out, accumulate=False))
         act = scratch_buf("moe.act", (T * self.top, self.F), self.dtype, dev)
         parts = scratch_buf("moe.parts", (T, self.top, self.hidden), torch.float32, dev)
         ops.moe_experts(normed, self.w_gate_up, self.w_down, routing, self.top, act, parts, self.act, self.weight_on, self.limit,
@@ -282,8 +313,10 @@ class MoEFeedForward(Part):
             ops.moe_identity(stream if stream is not None else normed, routing, self.top, self.E, parts)
         if self.shared is None:
             return parts, None, None
-        shared_out = scratch_buf("moe.shared", (T, self.hidden), torch.float32, dev)
-        self.shared.forward(normed, shared_out, accumulate=False)
+        if side is None:
+            self.shared.forward(normed, shared_out, accumulate=False)
+        else:
+            side.join()
         # the gate's logit: whoever adds the terms takes its sigmoid
         return parts, shared_out, logits[:, self.n_out] if self.shared_gate_name else None
 
@@ -294,5 +327,5 @@ class MoEFeedForward(Part):
         ops.rmsnorm_add(parts, None, 0.0, residual, extra, gate, gate_sigmoid=True, accumulate=accumulate)
 
     def forward(self, normed: torch.Tensor, residual: torch.Tensor, accumulate: bool = True,
-                stream: Optional[torch.Tensor] = None, tokens: Optional[torch.Tensor] = None) -> None:
-        self.add_parts(self.forward_parts(normed, stream, tokens), residual, accumulate)
+                stream: Optional[torch.Tensor] = None, step=None) -> None:
+        self.add_parts(self.forward_parts(normed, stream, step), residual, accumulate)

@@ -293,6 +293,8 @@ class AttentionMixer(Part):
         holds at most that many SMs (a block that runs another mixer beside this one leaves it the rest)."""
         T = step.n_rows
         kv = cache.kv[self.cache_key]
+        if self._prepares_at_once(qkv, cache):
+            return self._mix_prepared(qkv, step, cache, kv, out, max_blocks)
         projected = qkv                    # (the gate's columns stay there)
         if self.conv_taps:
             qkv = self._convolved(qkv, step, cache)
@@ -333,6 +335,44 @@ class AttentionMixer(Part):
                       max_blocks, softcap=self.softcap, sink=self.sink, keep_first=self.keep_first, sink_values=self.sink_values,
                       chunk=self.chunk, head_gate=head_gate)
         return self._joined(self._gated(att, projected), joined)
+
+    def _prepares_at_once(self, qkv: torch.Tensor, cache: LayerCache) -> bool:
+        """Whether convolution, norm, rotation and stores run as one kernel: one map, values of their own that are not blended, no
+        norm per head, neighbouring pairs (or no rotation), and something in front of the stores that the attention kernels do
+        not do themselves."""
+        table = self.position.rotation_table()
+        return (qkv.is_cuda and self.maps == 1 and self.values == "projection" and self.v_mix is None and self.head_norm is None
+                and self.qk_norm_eps is None and table is not None and cache.writes and cache.kv_writes
+                and (table.numel() == 0 or getattr(self.position, "layout", "split_half") == "interleaved")
+                and (self.conv_taps > 0 or self.whole_norm is not None)
+                and ops.qkv_prepare_ok(self.H, self.KV, self.hd, max(1, self.conv_taps), qkv.stride(0) if qkv.shape[0] > 1 else qkv.shape[1],
+                                       self.q_off))
+
+    def _mix_prepared(self, qkv: torch.Tensor, step: StepInfo, cache: LayerCache, kv, out: Optional[torch.Tensor], max_blocks: int) -> torch.Tensor:
+        T, H, KV, hd = step.n_rows, self.H, self.KV, self.hd
+        buf = lambda tag, shape, dt: scratch_buf(f"attention.{self.cache_key}.{tag}", shape, dt, qkv.device)
+        more = dict(taps=self.conv_w, state=cache.state.get(self.cache_key + ".conv")) if self.conv_taps else {}
+        if self.whole_norm:
+            more.update(q_weight=self.q_norm_w, k_weight=self.k_norm_w, eps=float(self.whole_norm["eps"]), q_count=H * self.qk_dim,
+                        k_count=KV * self.qk_dim)
+        args = (qkv, self.q_off, H, KV, hd, self.position.rotation_table(), float(getattr(self.position, "amplitude", 1.0)), step)
+        head_gate = qkv[:, self.g_off:self.g_off + self.Hq] if self.gate and self.gate_per == "head" else None
+        att = out if out is not None else buf("out", (T, H * hd), self.dtype)
+        same = dict(softcap=self.softcap, sink=self.sink, keep_first=self.keep_first, sink_values=self.sink_values, chunk=self.chunk,
+                    head_gate=head_gate)
+        if step.max_new == 1 and ops.attention_decode_fused_ok(qkv, self.dtype, H, KV, hd):
+            ready = buf("ready", (T, self.conv_channels), torch.float32)
+            ops.qkv_prepare(*args, out=ready, **more)
+            ops.attention_decode_fused(ready, 0, H * hd, (H + KV) * hd, kv.k_pages, kv.v_pages, self._no_rotation, True, kv.block_table,
+                                       step.positions, step.row_seq, step.slots, att, H, KV, hd, self.scale, self.window or 0,
+                                       step.max_context, self._arrivals, **same)
+        else:
+            q = buf("q", (T, H * hd), self.dtype)
+            ops.qkv_prepare(*args, q_out=q, k_pages=kv.k_pages, v_pages=kv.v_pages, block_table=kv.block_table, **more)
+            ops.attention(q, kv.k_pages, kv.v_pages, kv.block_table, step.positions, step.row_seq, step.slots, att, H, KV, hd, self.scale,
+                          self.window or 0, step.max_context if step.max_new == 1 else 0, step.cu_seqlens, step.start_pos, step.max_context,
+                          max_blocks, **same)
+        return self._gated(att, qkv)
 
     def _convolved(self, qkv: torch.Tensor, step: StepInfo, cache: LayerCache) -> torch.Tensor:
         """The convolved q | k | v columns, the values blended with the group's first layer's, float32 [T, q | k | v].  The first

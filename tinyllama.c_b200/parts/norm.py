@@ -42,11 +42,13 @@ class RMSNorm(Part):
         return out
 
     def add_normed(self, parts: Optional[torch.Tensor], residual: torch.Tensor, extra: Optional[torch.Tensor] = None,
-                   gate: Optional[torch.Tensor] = None, copy: Optional[torch.Tensor] = None) -> None:
+                   gate: Optional[torch.Tensor] = None, copy: Optional[torch.Tensor] = None,
+                   next_norm: Optional["RMSNorm"] = None) -> None:
         """As a sublayer's output norm: residual += norm(y) with y = the sum of parts [T, (n,) D] (+ sigmoid(gate[t]) *
         extra[t], gate being a logit per row).  copy [T, D]: receives the new residual rows in its own type (what the
-        next sublayer reads where it has no norm in front)."""
-        ops.rmsnorm_add(parts, self.weight, self.eps, residual, extra, gate, gate_sigmoid=True, copy=copy)
+        next sublayer reads where it has no norm in front), or with next_norm that norm of them (what it reads behind one)."""
+        ops.rmsnorm_add(parts, self.weight, self.eps, residual, extra, gate, gate_sigmoid=True, copy=copy,
+                        next_weight=None if next_norm is None else next_norm.weight, next_eps=0.0 if next_norm is None else next_norm.eps)
 
 
 @register_norm("layernorm")
