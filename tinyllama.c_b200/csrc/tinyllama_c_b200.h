@@ -349,13 +349,14 @@ int tlc_qk_whole_norm(float* qkv, int ld, int q_off, int q_n, const float* qw, i
  * neither; q_count, k_count: how many columns hold values), a rotation of neighbouring pairs of every query and key head's
  * first `rot` dimensions (cosines and sines times amplitude), then either out float [T, C], or q_out [T, H * hd] and the pages
  * of keys and values, of `dtype`.  single_rows: every sequence brings one row; all_fresh: every sequence starts at
- * position 0. */
+ * position 0.  sums: scratch of T * 2 * tlc_qkv_prepare_sums(...) floats (NULL without norms or with single rows). */
 int tlc_qkv_prepare_ok(int H, int KV, int hd, int K, int ld, int off);
 int tlc_qkv_prepare(const float* proj, int ld, int off, const float* w, int K, float* state, const float* q_w, const float* k_w,
                     int q_count, int k_count, float eps, const float* inv_freq, int rot, float amplitude, const int* positions,
                     const int* row_seq, const int* cu_seqlens, const int* slots, const int* start_pos, const int* block_table,
                     int max_pages, float* out, void* q_out, void* k_pages, void* v_pages, int dtype, int T, int B, int H, int KV,
-                    int hd, int single_rows, int all_fresh, cudaStream_t stream);
+                    int hd, int single_rows, int all_fresh, float* sums, cudaStream_t stream);
+int tlc_qkv_prepare_sums(int H, int KV, int hd);
 
 /* ---- gated delta rule (delta_rule.cu) -------------------------------------------------------------------
  * Per head: M <- a M; w = b (v - M^T k); M <- M + k w^T; r = M^T q (a the decay, b the write strength `beta`), with M

@@ -100,8 +100,9 @@ _SIGNATURES = {
     "tlc_softcap": (_i, [_vp, _ll, _f, _vp]),
     "tlc_rmsnorm_mean_add": (_i, [_vp, _i, _vp, _f, _f, _vp, _f, _i, _i, _vp, _i, _vp, _i, _vp]),
     "tlc_qkv_prepare_ok": (_i, [_i, _i, _i, _i, _i, _i]),
+    "tlc_qkv_prepare_sums": (_i, [_i, _i, _i]),
     "tlc_qkv_prepare": (_i, [_vp, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _f, _vp, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp,
-                             _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp]),
+                             _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp]),
     "tlc_qk_whole_norm": (_i, [_vp, _i, _i, _i, _vp, _i, _i, _vp, _f, _i, _i, _i, _vp]),
     "tlc_shift_mix": (_i, [_vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp]),
     "tlc_wkv_scan": (_i, [_vp, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _i, _vp]),
@@ -1326,7 +1327,7 @@ def qkv_prepare(proj: torch.Tensor, off: int, H: int, KV: int, hd: int, inv_freq
                 k_weight: Optional[torch.Tensor] = None, eps: float = 0.0, q_count: Optional[int] = None, k_count: Optional[int] = None,
                 out: Optional[torch.Tensor] = None, q_out: Optional[torch.Tensor] = None, k_pages: Optional[torch.Tensor] = None,
                 v_pages: Optional[torch.Tensor] = None, block_table: Optional[torch.Tensor] = None) -> None:
-    """In one kernel, on the columns queries | keys | values from `off` of the float32 projection proj [T, *] (H, KV and KV
+    """At once (single-token steps: in one kernel; prompts: in one more for the norms' sums), on the columns queries | keys | values from `off` of the float32 projection proj [T, *] (H, KV and KV
     heads of hd): the convolution over time (taps float32 [K, C], state as in channel_conv; None: none), the norms over all
     query and all key columns (weights float32, both or neither; q_count, k_count as in qk_whole_norm), the rotation of
     neighbouring pairs by position * inv_freq[i] with cosines and sines times amplitude, and then out float32 [T, C], or (out
@@ -1354,13 +1355,17 @@ def qkv_prepare(proj: torch.Tensor, off: int, H: int, KV: int, hd: int, inv_freq
             raise KernelError("qkv_prepare: q_out [T, H*hd] and pages [n, KV, 64, hd] contiguous and of one type")
     global _launches
     fresh, single = _all_fresh(step), int(step.max_new == 1)
-    if K > 1 and not fresh and not (single and T == step.n_seqs):
-        _launches += 1                  # (the kept rows are written by a kernel of their own)
+    single_kernel = single and T == step.n_seqs
+    sums = None
+    if not single_kernel and q_weight is not None:
+        sums = torch.empty((T, 2 * library().tlc_qkv_prepare_sums(H, KV, hd)), dtype=torch.float32, device=proj.device)
+    if not single_kernel:               # (the sums' kernel; the one that writes the kept rows)
+        _launches += int(sums is not None) + int(K > 1 and not fresh)
     _call("tlc_qkv_prepare", proj.data_ptr(), ld, int(off), _p(taps), K, _window(state, K, C, "qkv_prepare"), _p(q_weight), _p(k_weight),
           int(q_count or H * hd), int(k_count or KV * hd), float(eps), inv_freq.data_ptr(), 2 * inv_freq.numel(), float(amplitude),
           step.positions.data_ptr(), step.row_seq.data_ptr(), step.cu_seqlens.data_ptr(), step.slots.data_ptr(), step.start_pos.data_ptr(),
           _p(block_table), 0 if block_table is None else block_table.shape[1], _p(out), _p(q_out), _p(k_pages), _p(v_pages), dtype, T,
-          step.n_seqs, H, KV, hd, single, fresh, _stream())
+          step.n_seqs, H, KV, hd, single, fresh, _p(sums), _stream())
 
 
 # ---- time mixing with a decaying matrix state -------------------------------------------------------------------
