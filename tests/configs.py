@@ -445,8 +445,8 @@ def _fob_moe(experts, top, ff, limit, shared=None):
 # positions and none; keys wider and narrower than values, one head per key head, six on one, two, four and one taps; a ramp, plain
 # frequencies and no rotation at all; latents of 20 and 33 values (no tensor-core kernel), two thirds of the rotated part
 # rotated; every expert chosen, a single expert, one chosen of five; with and without a shared expert; a layer without
-# feed-forward
-FOBATAR_A = dict(architecture="Fobatar", vocab=150, width=52, embedding=dict(scale=3.0), norm=dict(eps=1e-5), residual_mult=0.6,
+# feed-forward; an embedding scale small enough that what is generated varies (the head is the embedding)
+FOBATAR_A = dict(architecture="Fobatar", vocab=150, width=52, embedding=dict(scale=0.8), norm=dict(eps=1e-5), residual_mult=0.6,
                  loop=dict(start=0, stop=2, times=3), layers=[
     _fob_att(4, 2, 24, 16, 2, 0.3, _k_rot(100.0, 8, factor=4.0, original=64, fast=8.0, slow=2.0), 5, _fob_moe(4, 2, 20, 1.0, shared=(12, 0.7))),
     _fob_lat(3, 10, 6, 14, 20, 0.25, _k_rot(10000.0, 4), None),
@@ -458,7 +458,7 @@ FOBATAR_A = dict(architecture="Fobatar", vocab=150, width=52, embedding=dict(sca
 # B: heads of 64 and of 128 (the tcgen05 attention of prompts, the one-kernel attention of single tokens) in chunks of 100, of
 # 33 and of exactly a page, values narrower than keys, three to five taps; latents of 48 and 80 values behind rotated parts of 16
 # and 32 (the tensor-core kernel); the repeated range in the middle, twice; latent attention first
-FOBATAR_B = dict(architecture="Fobatar", vocab=97, width=64, embedding=dict(scale=5.0), norm=dict(eps=1e-6), residual_mult=0.8,
+FOBATAR_B = dict(architecture="Fobatar", vocab=97, width=64, embedding=dict(scale=0.6), norm=dict(eps=1e-6), residual_mult=0.8,
                  loop=dict(start=1, stop=3, times=2), layers=[
     _fob_lat(4, 16, 16, 24, 48, 0.18, _k_rot(10000.0, 16, factor=4.0, original=64, fast=8.0, slow=1.0), _fob_moe(6, 2, 32, 1.0, shared=(16, 2.0))),
     _fob_att(4, 2, 64, 64, 3, 0.11, _k_rot(50000.0, 32, factor=2.0, original=100, fast=16.0, slow=1.0), 100,
@@ -495,7 +495,7 @@ def fobatar_random(seed: int) -> dict:
         kv, dim = pick(1, 2, 3), pick(8, 10, 16, 24, 64, 128)
         layers.append(_fob_att(kv * pick(1, 2, 3, 5), kv, dim, pick(6, 8, 16, 20, 64), pick(1, 2, 3, 4, 6), float(dim ** -0.5 * rng.uniform(0.5, 2.0)),
                                _k_rot(base, pick(0, 2, dim // 4 * 2, dim), **(sc or {})), pick(None, 1, 7, 40, 64, 90), mlp))
-    cfg = dict(architecture="Fobatar", vocab=pick(50, 131, 300), width=pick(32, 44, 50, 64, 96), embedding=dict(scale=pick(1.0, 2.5, 8.0)),
+    cfg = dict(architecture="Fobatar", vocab=pick(50, 131, 300), width=pick(32, 44, 50, 64, 96), embedding=dict(scale=pick(0.5, 1.0, 8.0)),
                norm=dict(eps=pick(1e-5, 1e-6)), residual_mult=pick(0.5, 1.0, 1.3), layers=layers)
     if rng.random() < 0.7:
         start = int(rng.integers(0, len(layers)))

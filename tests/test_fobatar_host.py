@@ -30,7 +30,7 @@ def test_builder_names_shapes_and_cache_needs():
     specs = {s.name: s for s in m.weight_specs()}
     got = {n: tuple(s.shape) for n, s in specs.items()}
     assert got["embed"] == (150, 52) and got["final.norm"] == (52,) and "head" not in got and m.head_name is None
-    assert m.embed_scale == 3.0
+    assert m.embed_scale == 0.8
     # attention: four query heads of 24 on two key heads, values of 16, two taps on every channel, whole-projection norms, a gate row a head
     assert all(got[f"l0.{n}"] == (52,) for n in ("norm1", "norm1b", "norm2", "norm2b"))
     assert got["l0.mix.q"] == (96, 52) and got["l0.mix.k"] == (48, 52) and got["l0.mix.v"] == (32, 52) and got["l0.mix.o"] == (52, 64)

@@ -97,7 +97,7 @@ def test_chunks_and_head_gate_of_prompts_on_tcgen05(H, KV, hd, chunk, key_ranges
 
 
 @pytest.mark.parametrize("chunk", CHUNKS)
-@pytest.mark.parametrize("H,KV,hd,rope", [(8, 2, 128, 64), (6, 1, 64, 64), (6, 3, 64, 0), (2, 2, 256, 128)])
+@pytest.mark.parametrize("H,KV,hd,rope", [(8, 2, 128, 64), (6, 1, 64, 64), (4, 4, 64, 0), (2, 2, 256, 128)])
 def test_chunks_and_head_gate_of_single_tokens_in_one_kernel(H, KV, hd, rope, chunk):
     """Rotation, store of the new row and attention in one launch: the keys in one piece a block, in several pieces that another
     block merges, and pieces of two rounds."""
